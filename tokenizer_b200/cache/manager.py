@@ -2,11 +2,11 @@
 and slots for per-request state of fixed size.
 
 Calls of the model's order whose mixers need the same kind of storage (the
-same kv heads, head size, window and chunk size) form a *group*.  A group owns its pages
+same kv heads, head size, window, kept first tokens and chunk size) form a *group*.  A group owns its pages
 (an allocator and one device pool) and every request has one block table per
 group, because groups differ in what they keep: a group of all keys keeps every
 page of a request, a group with a window gives a page back as soon as the
-window has passed it, a group whose keys are read inside chunks as soon as a request's next
+window has passed it (the pages of a sequence's first tokens stay, where the window keeps those), a group whose keys are read inside chunks as soon as a request's next
 position lies in a later chunk.  Inside a group every call has its own layer of the pool,
 addressed by the same table.  Beside the pages the manager owns the state
 arenas: one tensor [state slots, *shape] per call whose mixer declares state;
@@ -32,6 +32,7 @@ class GroupLayout:
     window: Optional[int]
     planes: int = 2                                  # rows a token stores per call (keys and values, or one for both)
     chunk: Optional[int] = None                      # keys are read inside chunks of this many positions only
+    keep_first: int = 0                              # a sequence's first tokens, which no window or chunk passes
     calls: List[int] = field(default_factory=list)   # calls of the order that write here
 
     @property
@@ -66,12 +67,15 @@ def plan_groups(needs) -> (List[GroupLayout], List[Optional[int]]):
         if need is None or need.kv is None:
             group_of.append(None)
             continue
-        key = (need.kv.kv_heads, need.kv.head_dim, need.kv.window, need.kv.planes, need.kv.chunk)
+        key = (need.kv.kv_heads, need.kv.head_dim, need.kv.window, need.kv.planes, need.kv.chunk,
+               need.kv.keep_first)
         for g, layout in enumerate(groups):
-            if (layout.kv_heads, layout.head_dim, layout.window, layout.planes, layout.chunk) == key:
+            if (layout.kv_heads, layout.head_dim, layout.window, layout.planes, layout.chunk,
+                    layout.keep_first) == key:
                 break
         else:
-            groups.append(GroupLayout(need.kv.kv_heads, need.kv.head_dim, need.kv.window, need.kv.planes, need.kv.chunk))
+            groups.append(GroupLayout(need.kv.kv_heads, need.kv.head_dim, need.kv.window, need.kv.planes, need.kv.chunk,
+                                      need.kv.keep_first))
             g = len(groups) - 1
         groups[g].calls.append(call)
         group_of.append(g)
@@ -120,6 +124,16 @@ class CachePlan:
             first = max(first, position - position % chunk)      # the start of the position's own chunk
         return first // self.page_size
 
+    def kept_blocks(self, group: int, before: int) -> int:
+        """How many blocks in front of block `before` hold first tokens that stay readable for good."""
+        return min(pages_for(self.groups[group].keep_first, self.page_size), before)
+
+    def wanted_blocks(self, group: int, position: int, end_block: int):
+        """The logical blocks before `end_block` that a query at `position` or later can still read."""
+        first = self.first_needed_block(group, position)
+        yield from range(self.kept_blocks(group, min(first, end_block)))
+        yield from range(first, end_block)
+
     def pages_missing(self, cache: RequestCache, n_new: int) -> List[int]:
         """Per group, the pages a step of `n_new` more tokens still needs."""
         missing = []
@@ -131,9 +145,8 @@ class CachePlan:
                 # nothing is given back before the end): only blocks past its end are missing
                 missing.append(max(0, end_block - len(table)))
                 continue
-            first = self.first_needed_block(g, cache.length)
-            count = sum(1 for b in range(first, end_block) if b >= len(table) or table[b] < 0)
-            missing.append(count)
+            missing.append(sum(1 for b in self.wanted_blocks(g, cache.length, end_block)
+                               if b >= len(table) or table[b] < 0))
         return missing
 
     def can_reserve(self, cache: RequestCache, n_new: int) -> bool:
@@ -158,22 +171,22 @@ class CachePlan:
                 while len(table) < end_block:          # no holes below the table's end (see pages_missing)
                     table.append(allocator.take())
                 continue
-            first = self.first_needed_block(g, cache.length)
             while len(table) < end_block:
                 table.append(-1)
-            for b in range(first, end_block):
+            for b in self.wanted_blocks(g, cache.length, end_block):
                 if table[b] < 0:
                     table[b] = allocator.take()
 
     def commit(self, cache: RequestCache, n_new: int) -> None:
         """The step ran: the request now holds n_new more tokens.  Pages that
-        every later query's window has passed are given back."""
+        every later query's window has passed are given back, those of kept first tokens excepted."""
         cache.length += n_new
         for g, allocator in enumerate(self.allocators):
             if self.groups[g].keeps_all:
                 continue
             table = cache.tables[g]
-            for b in range(min(self.first_needed_block(g, cache.length), len(table))):
+            passed = min(self.first_needed_block(g, cache.length), len(table))
+            for b in range(self.kept_blocks(g, passed), passed):
                 if table[b] >= 0:
                     allocator.give_back(table[b])
                     table[b] = -1

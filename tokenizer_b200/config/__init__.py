@@ -4,11 +4,12 @@ from .registry import (config_class_for, config_from_dict, load_config, register
 from .qwen2 import Qwen2Config
 from .pufuzen import PufuzenConfig
 from .katopel import KatopelConfig
+from .kazepel import KazepelConfig
 from .vizonex import VizonexConfig
 from .zobelorn import ZobelornConfig
 
 __all__ = [
-    "ConfigError", "KatopelConfig", "LayerCall", "LayerSpec", "ModelSpec", "PartSpec", "PufuzenConfig", "Qwen2Config", "VizonexConfig", "ZobelornConfig",
+    "ConfigError", "KatopelConfig", "KazepelConfig", "LayerCall", "LayerSpec", "ModelSpec", "PartSpec", "PufuzenConfig", "Qwen2Config", "VizonexConfig", "ZobelornConfig",
     "config_class_for", "config_from_dict", "load_config", "register_architecture",
     "registered_architectures",
 ]

@@ -22,6 +22,10 @@
 // values per (row, head, split)); the block that finishes last for a (row, kv
 // head) merges them in index order and writes the output.
 //
+// `keep_first` (> 0): the sequence's first keys that stay visible although the window has passed them.  They
+// are the first keys of the row's walk: everything below counts in places of the walk (0 .. n_keys - 1), and
+// place i is key i for the kept ones and key lo + i - kept behind them.
+//
 // HEAD_DIM is a compile-time size (a multiple of 16, at most 256), given with
 // -DHEAD_DIM=...; the library is built per head size at first use.
 #include "common.cuh"
@@ -113,7 +117,7 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
                         const __nv_bfloat16* __restrict__ v_pool, __nv_bfloat16* __restrict__ out,
                         const int* __restrict__ block_table, int table_stride,
                         const int* __restrict__ row_req, const int* __restrict__ pos, int nh,
-                        int nkv, int page, int window, int key_chunk, float scale,
+                        int nkv, int page, int window, int key_chunk, int keep_first, float scale,
                         float* __restrict__ scratch, int* __restrict__ counters, int min_chunk,
                         const int* __restrict__ rows, const float* __restrict__ sink, float softcap) {
   extern __shared__ __align__(16) unsigned char dec_smem[];
@@ -127,14 +131,16 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
   const int row = rows ? rows[z] : z;
   const int r = row < 0 ? -1 : row_req[row];
   const int p = r < 0 ? 0 : pos[row];
-  const int lo = first_visible_key(p, window, key_chunk);
-  const int n_keys = p - lo + 1;
+  const int lo = first_key_with_kept(first_visible_key(p, window, key_chunk), keep_first);
+  const int kept = kept_first_keys(lo, keep_first);
+  const int n_keys = p - lo + 1 + kept;
+  auto key_at = [&](int place) { return place < kept ? place : lo + place - kept; };
   const int chunk = split_chunk(n_keys, min_chunk);
   const int n_splits = (n_keys + chunk - 1) / chunk;
   const bool idle = r < 0 || split >= n_splits;
   if (!idle) {
     // the block's table entries, into L1 for the lookups below
-    const int first_page = (lo + split * chunk) / page, last_page = min(p, lo + split * chunk + chunk - 1) / page;
+    const int first_page = key_at(max(split * chunk, min(kept, n_keys - 1))) / page, last_page = key_at(min(n_keys, split * chunk + chunk) - 1) / page;
     for (int e = first_page + (int)threadIdx.x * 32; e <= last_page; e += DEC_THREADS * 32)
       asm volatile("prefetch.global.L1 [%0];" ::"l"(block_table + (size_t)r * table_stride + e));
     // ... and the keys and values of the block's first pass towards L2: all but the row's newest
@@ -143,8 +149,9 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
     // slower (268 MB at 64 rows of 8,192 keys: 76 us against 68 without).
     {
       const int* tb = block_table + (size_t)r * table_stride;
-      const int k_first = lo + split * chunk, k_last = min(p, k_first + min(chunk, DEC_BLOCK_KEYS) - 1);
-      for (int key = k_first + (int)threadIdx.x; key <= k_last; key += DEC_THREADS) {
+      const int k_first = split * chunk, k_last = min(n_keys, k_first + min(chunk, DEC_BLOCK_KEYS)) - 1;
+      for (int place = k_first + (int)threadIdx.x; place <= k_last; place += DEC_THREADS) {
+        const int key = key_at(place);
         const size_t at = ((size_t)(tb[key / page] * page + key % page) * nkv + kvh) * HEAD_DIM;
 #pragma unroll
         for (int c = 0; c < HEAD_DIM; c += 64) {
@@ -155,8 +162,8 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
     }
   }
   const int group = nh / nkv;                       // <= DEC_MAX_GROUP, checked by the launcher
-  const int first = lo + split * chunk;
-  const int last = min(p, first + chunk - 1);
+  const int first = split * chunk;                  // places of the row's walk
+  const int last = min(n_keys, first + chunk) - 1;
   const int* table = block_table + (size_t)(r < 0 ? 0 : r) * table_stride;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, t = lane & 3;
@@ -174,8 +181,8 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
   // lane that looked it up.
   const int page_shift = (page & (page - 1)) == 0 ? __ffs(page) - 1 : -1;
   auto tile_slots = [&](int k0) {
-    const int key = k0 + lane;
-    if (key > last) return -1;
+    if (k0 + lane > last) return -1;
+    const int key = key_at(k0 + lane);
     const int pg = page_shift >= 0 ? key >> page_shift : key / page;
     return table[pg] * page + (key - pg * page);
   };
@@ -214,7 +221,7 @@ decode_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16
   int turn = 0, slots_now = -1;
   const int k_mine = first + warp * DEC_TILE;
   const bool have_tile = !idle && k_mine <= last;
-  const bool early = EARLY && have_tile && k_mine + DEC_TILE - 1 < p;
+  const bool early = EARLY && have_tile && k_mine + DEC_TILE < n_keys;
   if (early) {
     slots_now = tile_slots(k_mine);
     if (kVBuffers == 2) stage_values(slots_now, v_buf);
@@ -500,10 +507,10 @@ TOKB200_API int tokb200_decode_attention_head_dim() { return HEAD_DIM; }
 TOKB200_API int tokb200_decode_attention(
     const void* q, const void* k_pool, const void* v_pool, void* out, const int* block_table,
     int table_stride, const int* row_req, const int* pos, int n_rows, int nh, int nkv, int d,
-    int page, int window, int key_chunk, float scale, float* scratch, int* counters, const int* rows,
+    int page, int window, int key_chunk, int keep_first, float scale, float* scratch, int* counters, const int* rows,
     const float* sink, float softcap, cudaStream_t stream) {
   if (n_rows <= 0) return TOKB200_OK;
-  if (d != HEAD_DIM || nh <= 0 || nkv <= 0 || nh % nkv || nh / nkv > DEC_MAX_GROUP || page <= 0 ||
+  if (d != HEAD_DIM || nh <= 0 || nkv <= 0 || nh % nkv || nh / nkv > DEC_MAX_GROUP || page <= 0 || keep_first < 0 ||
       nkv > 65535 || n_rows > 65535)
     return TOKB200_BAD_SIZE;
   if (((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)out) & 15)
@@ -515,8 +522,8 @@ TOKB200_API int tokb200_decode_attention(
   // no row sees more keys than its table reaches (or its window holds), so no row has
   // more pieces than this; blocks beyond would only find that out and leave
   long long reach = (long long)table_stride * page;
-  if (window >= 0 && window + 1 < reach) reach = window + 1;
-  if (key_chunk > 0 && key_chunk < reach) reach = key_chunk;
+  if (window >= 0 && (long long)window + 1 + keep_first < reach) reach = (long long)window + 1 + keep_first;
+  if (key_chunk > 0 && (long long)key_chunk + keep_first < reach) reach = (long long)key_chunk + keep_first;
   // The shortest piece for this launch: the candidate (a whole number of passes of 256 keys)
   // with the least estimated time, from a block's fixed cost (3), 2 per pass of 256 keys at head
   // size 64 (in proportion for others), 3 for a merge across blocks, and as many waves as the
@@ -574,7 +581,7 @@ TOKB200_API int tokb200_decode_attention(
   // one pool read as keys and as values, while a warp has two staging buffers (see ALIAS)
   const bool alias = k_pool == v_pool && kVBuffers == 2;
   void (*kernel)(const __nv_bfloat16*, const __nv_bfloat16*, const __nv_bfloat16*, __nv_bfloat16*, const int*,
-                 int, const int*, const int*, int, int, int, int, int, float, float*, int*, int, const int*,
+                 int, const int*, const int*, int, int, int, int, int, int, float, float*, int*, int, const int*,
                  const float*, float) =
       alias ? (early ? (cluster ? decode_attention_kernel<true, true, true> : decode_attention_kernel<false, true, true>)
                      : (cluster ? decode_attention_kernel<true, false, true> : decode_attention_kernel<false, false, true>))
@@ -595,7 +602,7 @@ TOKB200_API int tokb200_decode_attention(
     return launch_dependent(kernel, grid, dim3(DEC_THREADS), smem, stream,
                             (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pool,
                             (const __nv_bfloat16*)v_pool, (__nv_bfloat16*)out, block_table,
-                            table_stride, row_req, pos, nh, nkv, page, window, key_chunk, scale, scratch,
+                            table_stride, row_req, pos, nh, nkv, page, window, key_chunk, keep_first, scale, scratch,
                             counters, min_chunk, rows, sink, softcap);
   cudaLaunchConfig_t config = {};
   config.gridDim = grid;
@@ -617,7 +624,7 @@ TOKB200_API int tokb200_decode_attention(
   config.numAttrs = 2;
   cudaError_t err = cudaLaunchKernelEx(&config, kernel, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pool,
                                        (const __nv_bfloat16*)v_pool, (__nv_bfloat16*)out, block_table,
-                                       table_stride, row_req, pos, nh, nkv, page, window, key_chunk, scale, scratch,
+                                       table_stride, row_req, pos, nh, nkv, page, window, key_chunk, keep_first, scale, scratch,
                                        counters, min_chunk, rows, sink, softcap);
   return err == cudaSuccess ? TOKB200_OK : (int)err;
 }

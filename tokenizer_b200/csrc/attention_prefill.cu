@@ -13,6 +13,9 @@
 // is a multiple of 16).  A row's arithmetic depends on its position, its window
 // and its place in its 64-row tile only.
 //
+// `keep_first` (> 0): the sequence's first keys that stay visible although the window has passed them; the
+// blocks that hold them are walked in front of the others.
+//
 // HEAD_DIM is a compile-time size (multiple of 16, at most 128), -DHEAD_DIM=...
 #include "common.cuh"
 
@@ -71,15 +74,15 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 // share a key: one look-up in the block table serves the key's and the value's row.
 // The look-up (a dependent load) is made one block ahead of the copies that use it,
 // so the copies of a block are issued without waiting.  Keys outside [first_ok,
-// last_ok] are zero-filled and their pages are not touched (offset -1).
+// last_ok] and not among the kept first ones are zero-filled and their pages are not touched (offset -1).
 // The page of this thread's key in the block starting at key0 (-1: the key is not to
 // be read).  Only the load is issued here; `kv_row_offset` turns it into an offset
 // when the copies are issued, one block later, so nothing waits for the load.
 __device__ __forceinline__ int kv_page(const int* __restrict__ table, int page, int key0, int first_ok,
-                                       int last_ok) {
+                                       int last_ok, int keep_first) {
   static_assert(PF_THREADS == 2 * PF_KEYS && kChunks % 2 == 0, "two threads a key");
   const int key = key0 + (threadIdx.x >> 1);
-  if (key < first_ok || key > last_ok) return -1;
+  if ((key < first_ok && key >= keep_first) || key > last_ok) return -1;
   return table[key / page];
 }
 __device__ __forceinline__ long long kv_row_offset(int pg, int page, int nkv, int kvh, int key0) {
@@ -106,7 +109,7 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
                          const int* __restrict__ block_table, int table_stride,
                          const int* __restrict__ row_req, const int* __restrict__ pos,
                          const int* __restrict__ tiles, int n_tiles, int nh, int nkv, int page,
-                         int window, int chunk, float scale_log2, const float* __restrict__ sink,
+                         int window, int chunk, int keep_first, float scale_log2, const float* __restrict__ sink,
                          float cap_in, float cap_out) {
   extern __shared__ __align__(16) __nv_bfloat16 smem[];
   __nv_bfloat16* q_s = smem;                       // [64][kStride]
@@ -138,20 +141,23 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
     cp_async16(q_s + j * kStride + c * 8, src, ok);
   }
   const int kb_first = lo_first / PF_KEYS * PF_KEYS;
-  const int n_blocks = (pos_last - kb_first) / PF_KEYS + 1;
+  // blocks of kept keys that lie before the first block of the window
+  const int n_kept = min((keep_first + PF_KEYS - 1) / PF_KEYS, kb_first / PF_KEYS);
+  const int n_blocks = n_kept + (pos_last - kb_first) / PF_KEYS + 1;
+  auto first_of = [&](int b) { return b < n_kept ? b * PF_KEYS : kb_first + (b - n_kept) * PF_KEYS; };
   // fill the ring: blocks 0 .. PF_STAGES - 2 (q rides in the first group); a group is
   // committed for every block, existing or not, so that group counts stay in step
 #pragma unroll
   for (int b = 0; b < PF_STAGES - 1; ++b) {
     if (b < n_blocks) {
-      const int key0 = kb_first + b * PF_KEYS;
+      const int key0 = first_of(b);
       stage_kv(k_s + b * kTile, v_s + b * kTile, k_pool, v_pool,
-               kv_row_offset(kv_page(table, page, key0, lo_first, pos_last), page, nkv, kvh, key0));
+               kv_row_offset(kv_page(table, page, key0, lo_first, pos_last, keep_first), page, nkv, kvh, key0));
     }
     cp_async_commit();
   }
   int next_page = PF_STAGES - 1 < n_blocks
-      ? kv_page(table, page, kb_first + (PF_STAGES - 1) * PF_KEYS, lo_first, pos_last) : -1;
+      ? kv_page(table, page, first_of(PF_STAGES - 1), lo_first, pos_last, keep_first) : -1;
 
   // per thread: rows g and g + 8 of the warp's 16
   const int my_row[2] = {warp * 16 + g, warp * 16 + g + 8};
@@ -168,7 +174,7 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
   unsigned q_frag[HEAD_DIM / 16][4];
 
   for (int b = 0; b < n_blocks; ++b) {
-    const int kb = kb_first + b * PF_KEYS;
+    const int kb = first_of(b);
     const int stage = b % PF_STAGES;
     cp_async_wait<PF_STAGES - 2>();                 // block b has landed (for this thread)
     __syncthreads();                                // ... for all; and block b - 1 is no longer read
@@ -176,10 +182,10 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
       const int nb = b + PF_STAGES - 1;             // goes where block b - 1 was
       if (nb < n_blocks)
         stage_kv(k_s + (nb % PF_STAGES) * kTile, v_s + (nb % PF_STAGES) * kTile, k_pool, v_pool,
-                 kv_row_offset(next_page, page, nkv, kvh, kb_first + nb * PF_KEYS));
+                 kv_row_offset(next_page, page, nkv, kvh, first_of(nb)));
       cp_async_commit();
       next_page = nb + 1 < n_blocks
-          ? kv_page(table, page, kb_first + (nb + 1) * PF_KEYS, lo_first, pos_last) : -1;
+          ? kv_page(table, page, first_of(nb + 1), lo_first, pos_last, keep_first) : -1;
     }
     if (b == 0) {
 #pragma unroll
@@ -232,7 +238,7 @@ prefill_attention_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int key = kb + nt * 8 + 2 * t + (e & 1);
-          if (key > p_row[e >> 1] || key < lo_row[e >> 1]) s[nt][e] = -INFINITY;
+          if (key > p_row[e >> 1] || (key < lo_row[e >> 1] && key >= keep_first)) s[nt][e] = -INFINITY;
         }
       }
     }
@@ -328,10 +334,10 @@ TOKB200_API int tokb200_prefill_attention_head_dim() { return HEAD_DIM; }
 TOKB200_API int tokb200_prefill_attention(
     const void* q, const void* k_pool, const void* v_pool, void* out, const int* block_table,
     int table_stride, const int* row_req, const int* pos, const int* tiles, int n_tiles, int nh,
-    int nkv, int d, int page, int window, int chunk, float scale, const float* sink, float softcap,
+    int nkv, int d, int page, int window, int chunk, int keep_first, float scale, const float* sink, float softcap,
     cudaStream_t stream) {
   if (n_tiles <= 0) return TOKB200_OK;
-  if (d != HEAD_DIM || nh <= 0 || nkv <= 0 || nh % nkv || page <= 0 || nh > 65535)
+  if (d != HEAD_DIM || nh <= 0 || nkv <= 0 || nh % nkv || page <= 0 || nh > 65535 || keep_first < 0)
     return TOKB200_BAD_SIZE;
   if (((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)out) & 15)
     return TOKB200_BAD_ALIGNMENT;
@@ -350,6 +356,6 @@ TOKB200_API int tokb200_prefill_attention(
   prefill_attention_kernel<<<grid, PF_THREADS, smem, stream>>>(
       (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool,
       (__nv_bfloat16*)out, block_table, table_stride, row_req, pos, tiles, n_tiles, nh, nkv, page,
-      window, chunk, scale_log2, sink, softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap / scale : 0.f);
+      window, chunk, keep_first, scale_log2, sink, softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap / scale : 0.f);
   return tokb200_launch_status();
 }

@@ -29,6 +29,9 @@
 // one runs out an error flag is set and all roles fall through to the common exit,
 // where tensor memory is given back.
 //
+// `keep_first` (> 0): the sequence's first keys that stay visible although the window has passed them; the
+// blocks that hold them are walked in front of the others.
+//
 // HEAD_DIM is a compile-time size (64 or 128), -DHEAD_DIM=...
 #include <cuda.h>
 
@@ -201,7 +204,7 @@ attention_tcgen05_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
                          const int* __restrict__ block_table, int table_stride,
                          const int* __restrict__ row_req, const int* __restrict__ pos,
                          const int* __restrict__ tiles, int n_tiles, int nh, int nkv, int page, int window,
-                         int chunk, float scale_log2, const float* __restrict__ sink, float cap_in,
+                         int chunk, int keep_first, float scale_log2, const float* __restrict__ sink, float cap_in,
                          float cap_out) {
   extern __shared__ __align__(1024) unsigned char fa_raw[];      // swizzle atoms: 1024-byte aligned
   unsigned char* q_s = fa_raw;
@@ -237,7 +240,10 @@ attention_tcgen05_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
   const int lo_first = first_visible_key(pos0, window, chunk);
   const int lo_last = first_visible_key(pos_last, window, chunk);
   const int kb_first = lo_first / FA_KEYS * FA_KEYS;
-  const int n_blocks = live ? (pos_last - kb_first) / FA_KEYS + 1 : 0;
+  // blocks of kept keys that lie before the first block of the window
+  const int n_kept = min((keep_first + FA_KEYS - 1) / FA_KEYS, kb_first / FA_KEYS);
+  const int n_blocks = live ? n_kept + (pos_last - kb_first) / FA_KEYS + 1 : 0;
+  auto first_of = [&](int b) { return b < n_kept ? b * FA_KEYS : kb_first + (b - n_kept) * FA_KEYS; };
   const int* table = block_table + (size_t)(live ? r_id : 0) * table_stride;
   constexpr int kSoftmaxWarps = FA_SOFTMAX_THREADS / 32;
   constexpr int kMmaWarp = kSoftmaxWarps + FA_LOADER_THREADS / 32;
@@ -301,8 +307,8 @@ attention_tcgen05_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
       if (use > 0 && !__all_sync(0xffffffffu, fa_mbar_wait(&kv_empty[buf], (use - 1) & 1))) { ok = false; break; }   // a warp gives up together
 #pragma unroll
       for (int t = t0; t < FA_KEYS; t += FA_LOADER_THREADS) {
-        const int key = kb_first + b * FA_KEYS + t;
-        const bool in = key >= lo_first && key <= pos_last;
+        const int key = first_of(b) + t;
+        const bool in = (key >= lo_first || key < keep_first) && key <= pos_last;
         size_t offset = 0;
         if (in) offset = ((size_t)(table[key / page] * page + key % page) * nkv + kvh) * HEAD_DIM;
 #pragma unroll
@@ -375,7 +381,7 @@ attention_tcgen05_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
     float m_ref = -INFINITY, l_run = 0.f;     // reference maximum (raw score units) and running sum
     bool ok = true;
     for (int b = 0; b < n_blocks; ++b) {
-      const int kb = kb_first + b * FA_KEYS + split * kSplitKeys;
+      const int kb = first_of(b) + split * kSplitKeys;
       if (!__all_sync(0xffffffffu, fa_mbar_wait(&s_full[b & 1], (b >> 1) & 1))) { ok = false; break; }
 
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -394,7 +400,7 @@ attention_tcgen05_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
 #pragma unroll
         for (int j = 0; j < kSplitKeys; ++j) {
           const int key = kb + j;
-          s[j] = (key <= p_row && key >= lo_row) ? s[j] : -INFINITY;
+          s[j] = (key <= p_row && (key >= lo_row || key < keep_first)) ? s[j] : -INFINITY;
           m_blk = fmaxf(m_blk, s[j]);
         }
       } else {
@@ -534,10 +540,10 @@ TOKB200_API int tokb200_attention_tcgen05_error(void) {
 TOKB200_API int tokb200_attention_tcgen05(
     const void* q, const void* k_pool, const void* v_pool, void* out, const int* block_table,
     int table_stride, const int* row_req, const int* pos, const int* tiles, int n_tiles, int nh,
-    int nkv, int d, int page, int window, int chunk, float scale, const float* sink, float softcap,
+    int nkv, int d, int page, int window, int chunk, int keep_first, float scale, const float* sink, float softcap,
     cudaStream_t stream) {
   if (n_tiles <= 0) return TOKB200_OK;
-  if (d != HEAD_DIM || nh <= 0 || nkv <= 0 || nh % nkv || page <= 0)
+  if (d != HEAD_DIM || nh <= 0 || nkv <= 0 || nh % nkv || page <= 0 || keep_first < 0)
     return TOKB200_BAD_SIZE;
   if (((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)out) & 15)
     return TOKB200_BAD_ALIGNMENT;
@@ -561,7 +567,7 @@ TOKB200_API int tokb200_attention_tcgen05(
   return launch_ordered(false, attention_tcgen05_kernel, grid, dim3(FA_THREADS), (size_t)kFaSmem, stream,
                           (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pool,
                           (const __nv_bfloat16*)v_pool, (__nv_bfloat16*)out, block_table, table_stride,
-                          row_req, pos, tiles, n_tiles, nh, nkv, page, window, chunk,
+                          row_req, pos, tiles, n_tiles, nh, nkv, page, window, chunk, keep_first,
                           scale * 1.4426950408889634f, sink, softcap > 0.f ? scale / softcap : 0.f,
                           softcap > 0.f ? softcap / scale : 0.f);
 }

@@ -173,6 +173,13 @@ __device__ __forceinline__ int first_visible_key(int p, int window, int chunk) {
   return lo;
 }
 
+// How many of a sequence's first `keep_first` keys lie before everything else the query sees, its first
+// other key being `lo`: such keys stay visible although the window has passed them (0 where there is no gap).
+__device__ __forceinline__ int kept_first_keys(int lo, int keep_first) { return lo > keep_first ? keep_first : 0; }
+// The query's first key once the kept ones that touch its window are counted in (a window that still reaches
+// them sees everything from 0 on).
+__device__ __forceinline__ int first_key_with_kept(int lo, int keep_first) { return lo > keep_first ? lo : 0; }
+
 // Scores squashed into (-cap, cap) before the softmax: cap * tanh(score / cap).  The kernels on tensor
 // cores keep raw products q . k and fold the score's scale into the exponential, so they squash the raw
 // product: softcap_raw(raw, scale / cap, cap / scale) times the scale is cap * tanh(raw * scale / cap).

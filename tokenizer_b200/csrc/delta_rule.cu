@@ -21,7 +21,7 @@
 //                    the lanes gathering one sum, the other half the other.  Tokens are staged through
 //                    shared memory in runs by a warp of its own (cp.async), a run ahead of the warps
 //                    that compute; a token's operands are in registers before the token before it is done
-//   gdn_out_norm     a warp a (token, head): o / rms(o) * gain * scale * silu(gate)
+//   gdn_out_norm     a warp a (token, head): o / rms(o) * gain * scale * silu(gate), or sigmoid(gate)
 #include "common.cuh"
 
 #define GDN_MAX_TAPS 16
@@ -637,10 +637,14 @@ gdn_step_kernel(const TI* __restrict__ proj, int ld, int qkv_at, int b_at, int a
   }
 }
 
+// silu, or the sigmoid alone
+__device__ __forceinline__ float gdn_gate(float z, int plain) { return plain ? gdn_sigmoid(z) : z * gdn_sigmoid(z); }
+
 template <typename TG, typename TO>
 __global__ void gdn_out_norm_kernel(const float* __restrict__ o, const TG* __restrict__ gate, int ld, int g_at,
                                     const float* __restrict__ gain, float scale, float eps, TO* __restrict__ out,
-                                    int n_rows, int heads, int vdim, const int* __restrict__ row_req) {
+                                    int n_rows, int heads, int vdim, const int* __restrict__ row_req,
+                                    int plain) {
   pdl_wait();
   pdl_launch();
   const int unit = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -659,10 +663,10 @@ __global__ void gdn_out_norm_kernel(const float* __restrict__ o, const TG* __res
     const float4 w = *reinterpret_cast<const float4*>(gain + lane * 4);
     const float ss4 = warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w);
     const float inv4 = (1.0f / sqrtf(ss4 / 128.0f + eps)) * scale;
-    y[lane * 4] = from_float<TO>(v.x * inv4 * w.x * (z.x * gdn_sigmoid(z.x)));
-    y[lane * 4 + 1] = from_float<TO>(v.y * inv4 * w.y * (z.y * gdn_sigmoid(z.y)));
-    y[lane * 4 + 2] = from_float<TO>(v.z * inv4 * w.z * (z.z * gdn_sigmoid(z.z)));
-    y[lane * 4 + 3] = from_float<TO>(v.w * inv4 * w.w * (z.w * gdn_sigmoid(z.w)));
+    y[lane * 4] = from_float<TO>(v.x * inv4 * w.x * gdn_gate(z.x, plain));
+    y[lane * 4 + 1] = from_float<TO>(v.y * inv4 * w.y * gdn_gate(z.y, plain));
+    y[lane * 4 + 2] = from_float<TO>(v.z * inv4 * w.z * gdn_gate(z.z, plain));
+    y[lane * 4 + 3] = from_float<TO>(v.w * inv4 * w.w * gdn_gate(z.w, plain));
     return;
   }
   float ss = 0.f;
@@ -671,7 +675,7 @@ __global__ void gdn_out_norm_kernel(const float* __restrict__ o, const TG* __res
   const float inv = (1.0f / sqrtf(ss / (float)vdim + eps)) * scale;
   for (int l = lane; l < vdim; l += 32) {
     const float z = to_float(gates[l]);
-    y[l] = from_float<TO>(row[l] * inv * gain[l] * (z * gdn_sigmoid(z)));
+    y[l] = from_float<TO>(row[l] * inv * gain[l] * gdn_gate(z, plain));
   }
 }
 
@@ -825,14 +829,14 @@ TOKB200_API int tokb200_gdn_scan(const float* qkv, const float* bg, int groups, 
 
 TOKB200_API int tokb200_gdn_out_norm(const float* o, const void* gate, int gate_dtype, int ld, int g_at,
                                      const float* gain, float scale, float eps, void* out, int out_dtype, int n_rows,
-                                     int heads, int vdim, const int* row_req, cudaStream_t stream) {
+                                     int heads, int vdim, const int* row_req, int plain, cudaStream_t stream) {
   if (n_rows <= 0) return TOKB200_OK;
   if (heads <= 0 || vdim <= 0) return TOKB200_BAD_SIZE;
   const long long units = (long long)n_rows * heads;
   dim3 grid((unsigned)((units + 7) / 8)), block(256);
 #define LAUNCH(TG, TO)                                                                                       \
   return launch_dependent(gdn_out_norm_kernel<TG, TO>, grid, block, 0, stream, o, (const TG*)gate, ld, g_at, \
-                          gain, scale, eps, (TO*)out, n_rows, heads, vdim, row_req)
+                          gain, scale, eps, (TO*)out, n_rows, heads, vdim, row_req, plain)
   if (gate_dtype == TOKB200_F32 && out_dtype == TOKB200_F32) LAUNCH(float, float);
   if (gate_dtype == TOKB200_F32 && out_dtype == TOKB200_BF16) LAUNCH(float, __nv_bfloat16);
   if (gate_dtype == TOKB200_BF16 && out_dtype == TOKB200_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);

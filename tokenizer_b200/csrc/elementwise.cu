@@ -676,10 +676,11 @@ TOKB200_API int tokb200_silu_gate(const void* gu, void* out, int dtype, int n_to
 // looked up in its block table (pages were reserved ahead), and the id is
 // appended to `history[step, r]`; `step_counter` counts the steps.
 // ----------------------------------------------------------------------------
+#define ADVANCE_GROUPS 32
 struct AdvanceGroups {
-  int* slots[4];
-  const int* tables[4];
-  int widths[4];
+  int* slots[ADVANCE_GROUPS];
+  const int* tables[ADVANCE_GROUPS];
+  int widths[ADVANCE_GROUPS];
   int count;
 };
 
@@ -721,7 +722,7 @@ TOKB200_API int tokb200_advance_decode(int* ids, const int* drawn, int* pos, int
                                        int n_rows, int* history, int* step_counter,
                                        cudaStream_t stream) {
   if (n_rows <= 0) return TOKB200_OK;
-  if (n_groups < 0 || n_groups > 4) return TOKB200_BAD_SIZE;
+  if (n_groups < 0 || n_groups > ADVANCE_GROUPS) return TOKB200_BAD_SIZE;
   AdvanceGroups groups;
   groups.count = n_groups;
   for (int g = 0; g < n_groups; ++g) {

@@ -8,6 +8,11 @@
 //               index), zero elsewhere; share[t, experts] = sigmoid(the shared expert's gate logit)
 //   moe_gate    act[t, c] = f(gate[t, c]) * up[t, c] * share[t, expert of lane c], f the activation
 //
+// A third way (MOE_SCORE_SOFTMAX): s = the softmax over all router outputs, chosen like the sigmoid's.  For both,
+// a group's worth is the sum of its `worth` largest choice scores (1 or 2), and with `renormalize` the chosen
+// scores are divided by their sum + 1e-20.  `identity`: the last that many of the outputs that are chosen among
+// stand for the token's input itself; the sum of their shares is the row's last column.
+//
 // moe_route knows a second way to score and choose (`score` = MOE_SCORE_SIGMOID): scores s =
 // sigmoid(z); the CHOICE is made on s + correction (a learned number an expert, or none), and only
 // among the experts of the `keep` best of `groups` equal groups of neighbouring experts, a group's
@@ -20,12 +25,83 @@
 // f(share * gate) * (share * up), and the down product adds the experts up unweighted.
 #include "common.cuh"
 
-enum : int { MOE_SCORE_SOFTMAX_OF_CHOSEN = 0, MOE_SCORE_SIGMOID = 1 };
+enum : int { MOE_SCORE_SOFTMAX_OF_CHOSEN = 0, MOE_SCORE_SIGMOID = 1, MOE_SCORE_SOFTMAX = 2 };
 enum : int { MOE_SHARED_NONE = 0, MOE_SHARED_GATED = 1, MOE_SHARED_ONE = 2 };
 #define MOE_ACT_CLAMPED_SWISH TOKB200_ACT_COUNT
 
 #define MOE_MAX_EXPERTS 1024
 
+// the largest value and, among equals, the lowest index over a warp's lanes (index -1: nothing to offer)
+__device__ __forceinline__ void moe_warp_best(float& value, int& index) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float v = __shfl_xor_sync(0xffffffffu, value, o);
+    const int i = __shfl_xor_sync(0xffffffffu, index, o);
+    if (i >= 0 && (index < 0 || v > value || (v == value && i < index))) {
+      value = v;
+      index = i;
+    }
+  }
+}
+
+// One warp chooses: the `keep` groups of the largest worth, then the `top` experts of the largest choice score
+// inside them (ties: the lower index), and writes the token's row of shares.  z: the scores.  Lane l looks after
+// groups and experts l, l + 32, ...
+__device__ __forceinline__ void moe_choose(const float* z, const float* choice, float* group_worth, unsigned char* open,
+                                           float* out, int experts, int real, int identity, int top, int groups,
+                                           int keep, int worth, int renormalize, float scale, int columns, int lane) {
+  const int size = experts / groups;
+  if (keep < groups) {
+    for (int g = lane; g < groups; g += 32) {
+      float first = -INFINITY, second = -INFINITY;
+      for (int e = g * size; e < (g + 1) * size; ++e) {
+        const float c = choice[e];
+        if (c > first) { second = first; first = c; } else if (c > second) { second = c; }
+      }
+      group_worth[g] = worth > 1 && size > 1 ? first + second : first;
+      open[g] = 0;
+    }
+    for (int k = 0; k < keep; ++k) {
+      int best = -1;
+      float value = -INFINITY;
+      for (int g = lane; g < groups; g += 32)
+        if (!open[g] && (best < 0 || group_worth[g] > value)) { best = g; value = group_worth[g]; }
+      moe_warp_best(value, best);
+      if (best >= 0 && best % 32 == lane) open[best] = 1;
+    }
+    __syncwarp();
+  }
+  for (int c = lane; c < columns; c += 32) out[c] = 0.f;
+  unsigned taken = 0u;                                  // bit i: expert lane + 32 i
+  float sum = 0.f;
+  for (int k = 0; k < top; ++k) {
+    int best = -1;
+    float value = -INFINITY;
+    for (int e = lane, i = 0; e < experts; e += 32, ++i)
+      if (!((taken >> i) & 1u) && (keep == groups || open[e / size]) && (best < 0 || choice[e] > value)) {
+        best = e;
+        value = choice[e];
+      }
+    moe_warp_best(value, best);
+    if (best < 0) break;
+    sum += z[best];
+    if (best % 32 == lane) taken |= 1u << (best / 32);
+  }
+  const float factor = renormalize ? scale / (sum + 1e-20f) : scale;
+  float through = 0.f;                                  // the identity experts' shares
+  __syncwarp();
+  for (int e = lane, i = 0; e < experts; e += 32, ++i)
+    if ((taken >> i) & 1u) {
+      if (e < real) out[e] = z[e] * factor;
+      else through += z[e] * factor;
+    }
+  if (identity > 0) {
+    through = warp_sum(through);
+    if (lane == 0) out[columns - 1] = through;
+  }
+}
+
+// `experts` counts every router output that is chosen among, the `identity` last ones included.
 // h: the feed-forward's input [T, hidden] (float32, or its bfloat16 rounding); w: float32
 // [experts + shared, hidden], the router's rows and behind them the shared expert's gate row.
 // A block a token: its warps take the logits in turn (32-bit sums), thread 0 then chooses.
@@ -33,11 +109,14 @@ template <typename TI>
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const TI* __restrict__ h, const float* __restrict__ w, int hidden, int experts, int top,
                  int shared_mode, float* __restrict__ share, int score, const float* __restrict__ correction,
-                 int groups, int keep, float scale) {
+                 int groups, int keep, float scale, int identity, int worth, int renormalize) {
   __shared__ float z[MOE_MAX_EXPERTS + 1];
-  __shared__ float choice[MOE_MAX_EXPERTS];
+  __shared__ float choice[MOE_MAX_EXPERTS], group_worth[MOE_MAX_EXPERTS];
+  __shared__ float scratch[33];
+  __shared__ unsigned char open[MOE_MAX_EXPERTS];                  // groups whose experts may be chosen
   const int shared = shared_mode == MOE_SHARED_GATED ? 1 : 0;      // router rows behind the experts'
-  const int columns = experts + (shared_mode != MOE_SHARED_NONE ? 1 : 0);
+  const int real = experts - identity;
+  const int columns = real + (shared_mode != MOE_SHARED_NONE ? 1 : 0) + (identity > 0 ? 1 : 0);
   pdl_wait();
   pdl_launch();
   const int t = blockIdx.x;
@@ -71,61 +150,31 @@ moe_route_kernel(const TI* __restrict__ h, const float* __restrict__ w, int hidd
   }
   __syncthreads();
   float* out = share + (size_t)t * columns;
-  for (int e = threadIdx.x; e < experts; e += blockDim.x) {
-    out[e] = 0.f;
-    if (score == MOE_SCORE_SIGMOID) {
-      const float s = 1.0f / (1.0f + expf(-z[e]));
+  if (score != MOE_SCORE_SOFTMAX_OF_CHOSEN) {
+    float highest = 0.f, total = 1.f;
+    if (score == MOE_SCORE_SOFTMAX) {
+      float m = -INFINITY, sum = 0.f;
+      for (int e = threadIdx.x; e < experts; e += blockDim.x) m = fmaxf(m, z[e]);
+      highest = block_max(m, scratch);
+      for (int e = threadIdx.x; e < experts; e += blockDim.x) sum += expf(z[e] - highest);
+      total = block_sum(sum, scratch);
+    }
+    for (int e = threadIdx.x; e < experts; e += blockDim.x) {
+      const float s = score == MOE_SCORE_SOFTMAX ? expf(z[e] - highest) / total : 1.0f / (1.0f + expf(-z[e]));
       z[e] = s;
       choice[e] = s + (correction ? correction[e] : 0.f);
     }
-  }
-  __syncthreads();
-  if (threadIdx.x != 0) return;
-  if (score == MOE_SCORE_SIGMOID) {
-    // groups of neighbours: only the experts of the `keep` groups whose two largest choice scores
-    // add up to the most can be chosen (ties: the lower group, the lower expert)
-    const int size = experts / groups;
-    unsigned open[MOE_MAX_EXPERTS / 32];
-    for (int i = 0; i < (groups + 31) / 32; ++i) open[i] = 0u;
-    if (keep < groups) {
-      for (int k = 0; k < keep; ++k) {
-        int best = -1;
-        float worth = -INFINITY;
-        for (int g = 0; g < groups; ++g) {
-          if ((open[g >> 5] >> (g & 31)) & 1u) continue;
-          float first = -INFINITY, second = -INFINITY;
-          for (int e = g * size; e < (g + 1) * size; ++e) {
-            const float c = choice[e];
-            if (c > first) { second = first; first = c; } else if (c > second) { second = c; }
-          }
-          const float sum = size > 1 ? first + second : first;
-          if (best < 0 || sum > worth) { best = g; worth = sum; }
-        }
-        if (best < 0) break;
-        open[best >> 5] |= 1u << (best & 31);
-      }
-    }
-    unsigned taken[MOE_MAX_EXPERTS / 32];
-    for (int i = 0; i < (experts + 31) / 32; ++i) taken[i] = 0u;
-    for (int k = 0; k < top; ++k) {
-      int best = -1;
-      float value = -INFINITY;
-      for (int e = 0; e < experts; ++e) {
-        const int g = e / size;
-        if (keep < groups && !((open[g >> 5] >> (g & 31)) & 1u)) continue;
-        if (!((taken[e >> 5] >> (e & 31)) & 1u) && (best < 0 || choice[e] > value)) {
-          best = e;
-          value = choice[e];
-        }
-      }
-      if (best < 0) break;
-      taken[best >> 5] |= 1u << (best & 31);
-      out[best] = z[best] * scale;
-    }
-    if (shared_mode == MOE_SHARED_ONE) out[experts] = 1.0f;
-    if (shared_mode == MOE_SHARED_GATED) out[experts] = 1.0f / (1.0f + expf(-z[experts]));
+    __syncthreads();
+    if (warp != 0) return;
+    moe_choose(z, choice, group_worth, open, out, experts, real, identity, top, groups, keep, worth, renormalize, scale,
+               columns, lane);
+    if (lane == 0 && shared_mode == MOE_SHARED_ONE) out[real] = 1.0f;
+    if (lane == 0 && shared_mode == MOE_SHARED_GATED) out[real] = 1.0f / (1.0f + expf(-z[experts]));
     return;
   }
+  for (int e = threadIdx.x; e < experts; e += blockDim.x) out[e] = 0.f;
+  __syncthreads();
+  if (threadIdx.x != 0) return;
   unsigned taken[MOE_MAX_EXPERTS / 32];
   for (int i = 0; i < (experts + 31) / 32; ++i) taken[i] = 0u;
   float highest = 0.f, sum = 0.f;
@@ -166,7 +215,7 @@ __device__ __forceinline__ float moe_glu(int act, float g, float u, float limit,
 template <typename T>
 __global__ void moe_gate_kernel(const T* __restrict__ gu, const float* __restrict__ share, T* __restrict__ out,
                                 int inner, int experts, int ff, int shared, int act, size_t n, float limit,
-                                float shared_limit, float alpha, int on_input) {
+                                float shared_limit, float alpha, int on_input, int share_ld) {
   pdl_wait();
   pdl_launch();
   const size_t stride = (size_t)gridDim.x * blockDim.x;
@@ -174,7 +223,7 @@ __global__ void moe_gate_kernel(const T* __restrict__ gu, const float* __restric
     const size_t t = i / inner;
     const int c = (int)(i % inner);
     const int e = c < experts * ff ? c / ff : experts;
-    const float w = share[t * (experts + shared) + e];
+    const float w = share[t * share_ld + e];
     float value = 0.f;
     if (w != 0.f) {
       const float g = to_float(gu[t * 2 * inner + c]), u = to_float(gu[t * 2 * inner + inner + c]);
@@ -189,7 +238,7 @@ __global__ void moe_gate_kernel(const T* __restrict__ gu, const float* __restric
 __global__ void moe_gate_bf16x8_kernel(const __nv_bfloat16* __restrict__ gu, const float* __restrict__ share,
                                        __nv_bfloat16* __restrict__ out, int inner, int experts, int ff, int shared,
                                        int act, size_t n8, float limit, float shared_limit, float alpha,
-                                       int on_input) {
+                                       int on_input, int share_ld) {
   pdl_wait();
   pdl_launch();
   const size_t stride = (size_t)gridDim.x * blockDim.x;
@@ -198,7 +247,7 @@ __global__ void moe_gate_bf16x8_kernel(const __nv_bfloat16* __restrict__ gu, con
     const size_t t = i / per_row;
     const int c = (int)(i % per_row) * 8;
     const int e = c < experts * ff ? c / ff : experts;
-    const float w = share[t * (experts + shared) + e];
+    const float w = share[t * share_ld + e];
     uint4 packed = make_uint4(0u, 0u, 0u, 0u);
     if (w != 0.f) {
       const uint4 graw = *reinterpret_cast<const uint4*>(gu + t * 2 * inner + c);
@@ -223,28 +272,32 @@ __global__ void moe_gate_bf16x8_kernel(const __nv_bfloat16* __restrict__ gu, con
 
 TOKB200_API int tokb200_moe_route(const void* h, int h_dtype, const float* w, int hidden, int experts, int top,
                                   int shared, float* share, int n_rows, int score, const float* correction,
-                                  int groups, int keep, float scale, cudaStream_t stream) {
+                                  int groups, int keep, float scale, int identity, int worth, int renormalize,
+                                  cudaStream_t stream) {
   if (n_rows <= 0) return TOKB200_OK;
+  if (identity < 0 || (identity > 0 && score == MOE_SCORE_SOFTMAX_OF_CHOSEN) || worth < 1 || worth > 2 || experts <= 0)
+    return TOKB200_BAD_SIZE;
+  experts += identity;                 // all that a token chooses among
   if (hidden <= 0 || experts <= 0 || experts > MOE_MAX_EXPERTS || top <= 0 || top > experts ||
       shared < MOE_SHARED_NONE || shared > MOE_SHARED_ONE ||
-      (score != MOE_SCORE_SOFTMAX_OF_CHOSEN && score != MOE_SCORE_SIGMOID) || groups <= 0 || experts % groups ||
+      score < MOE_SCORE_SOFTMAX_OF_CHOSEN || score > MOE_SCORE_SOFTMAX || groups <= 0 || experts % groups ||
       keep <= 0 || keep > groups || (long long)keep * (experts / groups) < top)
     return TOKB200_BAD_SIZE;
   if (h_dtype == TOKB200_F32)
     return launch_dependent(moe_route_kernel<float>, dim3(n_rows), dim3(128), 0, stream, (const float*)h, w, hidden,
-                            experts, top, shared, share, score, correction, groups, keep, scale);
+                            experts, top, shared, share, score, correction, groups, keep, scale, identity, worth, renormalize);
   if (h_dtype == TOKB200_BF16)
     return launch_dependent(moe_route_kernel<__nv_bfloat16>, dim3(n_rows), dim3(128), 0, stream,
                             (const __nv_bfloat16*)h, w, hidden, experts, top, shared, share, score, correction, groups,
-                            keep, scale);
+                            keep, scale, identity, worth, renormalize);
   return TOKB200_BAD_DTYPE;
 }
 
 TOKB200_API int tokb200_moe_gate(const void* gu, const float* share, void* out, int dtype, int n_rows, int inner,
                                  int experts, int ff, int shared, int act, float limit, float shared_limit,
-                                 float alpha, int on_input, cudaStream_t stream) {
+                                 float alpha, int on_input, int share_ld, cudaStream_t stream) {
   if (n_rows <= 0) return TOKB200_OK;
-  if (inner <= 0 || experts <= 0 || ff <= 0 || (long long)experts * ff > inner || act < 0 || act > MOE_ACT_CLAMPED_SWISH ||
+  if (inner <= 0 || experts <= 0 || ff <= 0 || share_ld < experts + (shared ? 1 : 0) || (long long)experts * ff > inner || act < 0 || act > MOE_ACT_CLAMPED_SWISH ||
       (!shared && (long long)experts * ff != inner))
     return TOKB200_BAD_SIZE;
   const size_t n = (size_t)n_rows * inner;
@@ -252,16 +305,16 @@ TOKB200_API int tokb200_moe_gate(const void* gu, const float* share, void* out, 
   const dim3 grid((unsigned)(blocks < 8192 ? blocks : 8192));
   if (dtype == TOKB200_F32)
     return launch_dependent(moe_gate_kernel<float>, grid, dim3(256), 0, stream, (const float*)gu, share, (float*)out,
-                            inner, experts, ff, shared, act, n, limit, shared_limit, alpha, on_input);
+                            inner, experts, ff, shared, act, n, limit, shared_limit, alpha, on_input, share_ld);
   if (dtype == TOKB200_BF16 && inner % 8 == 0 && ff % 8 == 0 && (((uintptr_t)gu | (uintptr_t)out) & 15) == 0) {
     const size_t n8 = n / 8, blocks8 = (n8 + 255) / 256;
     return launch_dependent(moe_gate_bf16x8_kernel, dim3((unsigned)(blocks8 < 65535 ? blocks8 : 65535)), dim3(256), 0,
                             stream, (const __nv_bfloat16*)gu, share, (__nv_bfloat16*)out, inner, experts, ff, shared,
-                            act, n8, limit, shared_limit, alpha, on_input);
+                            act, n8, limit, shared_limit, alpha, on_input, share_ld);
   }
   if (dtype == TOKB200_BF16)
     return launch_dependent(moe_gate_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)gu,
                             share, (__nv_bfloat16*)out, inner, experts, ff, shared, act, n, limit, shared_limit, alpha,
-                            on_input);
+                            on_input, share_ld);
   return TOKB200_BAD_DTYPE;
 }

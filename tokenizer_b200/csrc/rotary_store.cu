@@ -2,7 +2,8 @@
 // stacked product: the projection's bias, the rotation of the leading `rot_dims` lanes of every query
 // and key head in the interleaved form (lane 2i pairs with lane 2i + 1; the pair (u, v) at position p
 // becomes (u cos a - v sin a, v cos a + u sin a), a = float32(p) * inv_freq[i], or, where the frequencies come
-// in 64-bit (`inv_freq64`), the 64-bit product brought into one turn before it is rounded), and the write of the
+// in 64-bit (`inv_freq64`), the 64-bit product brought into one turn before it is rounded; cosine and sine are
+// multiplied by `magnitude`, 1 for a plain rotation), and the write of the
 // token's keys and values into its cache slot.  Cache rows and query rows have `row` lanes a head,
 // row >= max(dim, vdim): keys and queries fill the first `dim` lanes, values the first `vdim`, the
 // rest is written as zero, so that kernels which take one head size serve both.
@@ -19,7 +20,7 @@
 // turned by the angle of frequency i).  `head_norm`: after the rotation every query head and every key
 // head is divided by its own root mean square over its `dim` lanes (`head_eps` inside the root, no gain).
 // A rotation turns pairs and leaves each pair's sum of squares as it was, so a head's mean square is
-// taken of its lanes before the rotation, a warp a head, and kept in shared memory.  A token's sines and
+// taken of its lanes before the rotation (`magnitude` is 1 then), a warp a head, and kept in shared memory.  A token's sines and
 // cosines are computed once a frequency into shared memory (every head turns by the same angles).  `kv_heads` = 0: the
 // projection holds queries only (a layer that reads another layer's cache): nothing is written but q_out.
 //
@@ -58,7 +59,7 @@ __global__ void qkv_rotate_store_kernel(const TI* __restrict__ proj, int ld, int
                                         T* __restrict__ k_pool, T* __restrict__ v_pool, int heads, int kv_heads,
                                         int dim, int vdim, int row, const float* __restrict__ q_gain,
                                         const float* __restrict__ k_gain, float eps, const float* __restrict__ temp,
-                                        int half_layout, int head_norm, float head_eps, int quads) {
+                                        int half_layout, int head_norm, float head_eps, int quads, float magnitude) {
   // shared memory: a token's cosines and sines, one pair a frequency (every head turns by the same
   // angles), then the heads' inverse root mean squares (with `head_norm`)
   extern __shared__ float shared[];
@@ -80,7 +81,10 @@ __global__ void qkv_rotate_store_kernel(const TI* __restrict__ proj, int ld, int
     } else {
       angle = (float)p * inv_freq[i];
     }
-    sincosf(angle, &sine[i], &cosine[i]);
+    float sn, cs;
+    sincosf(angle, &sn, &cs);
+    sine[i] = sn * magnitude;
+    cosine[i] = cs * magnitude;
   }
   pdl_wait();
   pdl_launch();
@@ -247,7 +251,7 @@ TOKB200_API int tokb200_qkv_rotate_store(const void* proj, int proj_dtype, int l
                                          int out_dtype, int n_rows, int heads, int kv_heads, int dim, int vdim,
                                          int row, const float* q_gain, const float* k_gain, float eps,
                                          const float* temp, int half_layout, int head_norm, float head_eps,
-                                         cudaStream_t stream) {
+                                         float magnitude, cudaStream_t stream) {
   if (n_rows <= 0) return TOKB200_OK;
   if (kv_heads == 0 && (slot != nullptr || k_gain != nullptr)) return TOKB200_BAD_SIZE;
   const size_t smem = (size_t)(rot_dims + (head_norm ? heads + kv_heads : 0)) * sizeof(float);
@@ -259,14 +263,14 @@ TOKB200_API int tokb200_qkv_rotate_store(const void* proj, int proj_dtype, int l
   const int quads = proj_dtype == TOKB200_F32 && dim % 4 == 0 && vdim % 4 == 0 && row % 4 == 0 && rot_dims % 8 == 0 &&
                     at % 4 == 0 && ld % 4 == 0 && (all & 15) == 0;
   if (heads <= 0 || kv_heads < 0 || dim <= 0 || vdim <= 0 || row < dim || row < vdim || rot_dims < 0 ||
-      rot_dims % 2 || rot_dims > dim || (rot_dims > 0 && inv_freq == nullptr && inv_freq64 == nullptr))
+      rot_dims % 2 || rot_dims > dim || (head_norm && magnitude != 1.0f) || (rot_dims > 0 && inv_freq == nullptr && inv_freq64 == nullptr))
     return TOKB200_BAD_SIZE;
 #define LAUNCH(TI, T)                                                                                         \
   return launch_dependent(qkv_rotate_store_kernel<TI, T>, dim3(n_rows), dim3(256), smem, stream,              \
                           (const TI*)proj, ld, at, bias, inv_freq, inv_freq64, rot_dims, pos, slot, row_req,  \
                           (T*)q_out,                                                                          \
                           (T*)k_pool, (T*)v_pool, heads, kv_heads, dim, vdim, row, q_gain, k_gain, eps, temp, \
-                          half_layout, head_norm, head_eps, quads)
+                          half_layout, head_norm, head_eps, quads, magnitude)
   if (proj_dtype == TOKB200_F32 && out_dtype == TOKB200_F32) LAUNCH(float, float);
   if (proj_dtype == TOKB200_F32 && out_dtype == TOKB200_BF16) LAUNCH(float, __nv_bfloat16);
   if (proj_dtype == TOKB200_BF16 && out_dtype == TOKB200_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);

@@ -316,10 +316,11 @@ def _sink(sink, nh):
 
 def paged_attention_generic(q, k_pool, v_pool, out, block_table, row_req, pos, nh, nkv, d, page,
                             window, scale, sink: Optional[torch.Tensor] = None, chunk: Optional[int] = None,
-                            softcap: Optional[float] = None) -> None:
+                            softcap: Optional[float] = None, keep_first: int = 0) -> None:
     """`softcap` (optional, in every attention kernel): a score s becomes softcap * tanh(s / softcap) before
     the softmax.  `chunk` (optional): keys are seen inside chunks of that many positions counted from 0 (a
-    query sees the keys of its own chunk up to itself).  `sink` (float32, one per query head): a score without key or value that counts once in
+    query sees the keys of its own chunk up to itself).  `keep_first` (in every attention kernel): the
+    sequence's first keys that stay visible although window or chunk have passed them.  `sink` (float32, one per query head): a score without key or value that counts once in
     the softmax's denominator, unscaled.  `v_pool` may be `k_pool` itself (values that are the
     leading lanes of the key rows)."""
     if d > 1024:
@@ -329,7 +330,7 @@ def paged_attention_generic(q, k_pool, v_pool, out, block_table, row_req, pos, n
     _check(_lib("attention_generic").tokb200_paged_attention_generic(
         _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _i(_tag(q)), _ptr(block_table),
         _i(block_table.shape[1]), _ptr(row_req), _ptr(pos), _i(q.shape[0]), _i(nh), _i(nkv),
-        _i(d), _i(page), _i(-1 if window is None else int(window)), _i(0 if chunk is None else int(chunk)), _f(scale), _sink(sink, nh), _f(softcap or 0.0), _stream()),
+        _i(d), _i(page), _i(-1 if window is None else int(window)), _i(0 if chunk is None else int(chunk)), _i(int(keep_first)), _f(scale), _sink(sink, nh), _f(softcap or 0.0), _stream()),
         "paged_attention")
 
 
@@ -372,8 +373,8 @@ def advance_decode(ids, drawn, pos, kv_len, row_req, slots, tables, page, histor
     """After a decoding step: the drawn ids become the next inputs and every
     row's position, stored length and cache slot move on by one (on the device)."""
     n = len(slots)
-    if n > 4:
-        raise ValueError("advance_decode handles up to four cache groups")
+    if n > 32:
+        raise ValueError("advance_decode handles up to 32 cache groups")
     slot_ptrs = (ctypes.c_void_p * max(n, 1))(*[t.data_ptr() for t in slots])
     table_ptrs = (ctypes.c_void_p * max(n, 1))(*[t.data_ptr() for t in tables])
     widths = (ctypes.c_int * max(n, 1))(*[t.shape[1] for t in tables])
@@ -393,7 +394,7 @@ def decode_attention_supported(nh: int, nkv: int, d: int) -> bool:
 
 def decode_attention(q, k_pool, v_pool, out, block_table, row_req, pos, nh, nkv, d, page, window,
                      scale, rows: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None,
-                     chunk: Optional[int] = None, softcap: Optional[float] = None) -> None:
+                     chunk: Optional[int] = None, softcap: Optional[float] = None, keep_first: int = 0) -> None:
     """Attention for rows of one token each (bfloat16): keys are split over
     blocks and merged; the scratch for the pieces is kept per (device, rows,
     heads, head size) and reused by every layer, which run one after another.  With `rows`
@@ -415,7 +416,7 @@ def decode_attention(q, k_pool, v_pool, out, block_table, row_req, pos, nh, nkv,
     _check(lib.tokb200_decode_attention(
         _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(block_table),
         _i(block_table.shape[1]), _ptr(row_req), _ptr(pos), _i(n_rows), _i(nh), _i(nkv), _i(d),
-        _i(page), _i(-1 if window is None else int(window)), _i(0 if chunk is None else int(chunk)), _f(scale), _ptr(scratch),
+        _i(page), _i(-1 if window is None else int(window)), _i(0 if chunk is None else int(chunk)), _i(int(keep_first)), _f(scale), _ptr(scratch),
         _ptr(counters), _ptr(rows), _sink(sink, nh), _f(softcap or 0.0), _stream()), "decode_attention")
 
 
@@ -545,7 +546,7 @@ def prefill_attention_supported(nh: int, nkv: int, d: int) -> bool:
 
 def prefill_attention(q, k_pool, v_pool, out, block_table, row_req, pos, tiles, n_tiles, nh, nkv,
                       d, page, window, scale, sink: Optional[torch.Tensor] = None, chunk: Optional[int] = None,
-                      softcap: Optional[float] = None) -> None:
+                      softcap: Optional[float] = None, keep_first: int = 0) -> None:
     """Attention for portions of prompts (bfloat16).  `tiles` is int32 [n, 2]:
     (first row, rows <= 64) of consecutive rows of one request."""
     if q.dtype != torch.bfloat16:
@@ -556,7 +557,7 @@ def prefill_attention(q, k_pool, v_pool, out, block_table, row_req, pos, tiles, 
     _check(lib.tokb200_prefill_attention(
         _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(block_table),
         _i(block_table.shape[1]), _ptr(row_req), _ptr(pos), _ptr(tiles), _i(n_tiles), _i(nh),
-        _i(nkv), _i(d), _i(page), _i(-1 if window is None else int(window)), _i(0 if chunk is None else int(chunk)), _f(scale), _sink(sink, nh),
+        _i(nkv), _i(d), _i(page), _i(-1 if window is None else int(window)), _i(0 if chunk is None else int(chunk)), _i(int(keep_first)), _f(scale), _sink(sink, nh),
         _f(softcap or 0.0), _stream()), "prefill_attention")
 
 
@@ -791,7 +792,7 @@ def attention_tcgen05_supported(nh: int, nkv: int, d: int) -> bool:
 
 def attention_tcgen05(q, k_pool, v_pool, out, block_table, row_req, pos, tiles, n_tiles, nh, nkv, d,
                       page, window, scale, sink: Optional[torch.Tensor] = None, chunk: Optional[int] = None,
-                      softcap: Optional[float] = None) -> None:
+                      softcap: Optional[float] = None, keep_first: int = 0) -> None:
     """Attention for portions of prompts on tcgen05 (bfloat16, head size 64 or 128).
     `tiles` is int32 [n, 2]: (first row, rows <= 128) of consecutive rows of one request."""
     if q.dtype != torch.bfloat16:
@@ -802,7 +803,7 @@ def attention_tcgen05(q, k_pool, v_pool, out, block_table, row_req, pos, tiles, 
     _check(lib.tokb200_attention_tcgen05(
         _ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(out), _ptr(block_table),
         _i(block_table.shape[1]), _ptr(row_req), _ptr(pos), _ptr(tiles), _i(n_tiles), _i(nh),
-        _i(nkv), _i(d), _i(page), _i(-1 if window is None else int(window)), _i(0 if chunk is None else int(chunk)), _f(scale), _sink(sink, nh),
+        _i(nkv), _i(d), _i(page), _i(-1 if window is None else int(window)), _i(0 if chunk is None else int(chunk)), _i(int(keep_first)), _f(scale), _sink(sink, nh),
         _f(softcap or 0.0), _stream()), "attention_tcgen05")
 
 
@@ -1240,21 +1241,138 @@ def gdn_step(proj: torch.Tensor, qkv_at: int, b_at: int, a_at: int, g_at: int, g
 
 
 def gdn_out_norm(o: torch.Tensor, gate: torch.Tensor, g_at: int, gain: torch.Tensor, scale: float, eps: float,
-                 out: torch.Tensor, heads: int, vdim: int, row_req) -> None:
-    """out[t, h] = o[t, h] / sqrt(mean(o[t, h]^2) + eps) * gain * scale * silu(gate[t, g_at + h vdim ..])."""
+                 out: torch.Tensor, heads: int, vdim: int, row_req, gate_kind: str = "silu") -> None:
+    """out[t, h] = o[t, h] / sqrt(mean(o[t, h]^2) + eps) * gain * scale * silu(gate[t, g_at + h vdim ..]), or the
+    sigmoid of the gate (`gate_kind` "sigmoid")."""
+    if gate_kind not in ("silu", "sigmoid"):
+        raise ValueError("gdn_out_norm: the gate is silu or sigmoid")
     n = o.shape[0]
     if o.dtype != torch.float32 or tuple(o.shape) != (n, heads * vdim) or tuple(out.shape) != (n, heads * vdim) or \
             gain.numel() != vdim or g_at + heads * vdim > gate.shape[1]:
         raise ValueError("gdn_out_norm: o float32 [T, heads * vdim], a gain of vdim, the gate's columns inside its matrix")
     _check(_lib("delta_rule").tokb200_gdn_out_norm(
         _ptr(o), _sliced_ptr(gate), _i(_tag(gate)), _i(_ld(gate)), _i(g_at), _ptr(gain), _f(scale), _f(eps), _ptr(out),
-        _i(_tag(out)), _i(n), _i(heads), _i(vdim), _ptr(row_req), _stream()), "gdn_out_norm")
+        _i(_tag(out)), _i(n), _i(heads), _i(vdim), _ptr(row_req), _i(int(gate_kind == "sigmoid")), _stream()),
+        "gdn_out_norm")
+
+
+# ---- the delta rule with a decay a key channel ----
+CDR_RUN = 4        # tokens of a run (csrc/channel_delta.cu)
+
+
+def cdr_padded_dim(dim: int) -> int:
+    """Rows of a head's state column as the recurrence keeps it; 0: a size it does not take."""
+    return int(_lib("channel_delta").tokb200_cdr_padded_dim(_i(dim)))
+
+
+def cdr_record(dim: int, vdim: int) -> int:
+    """Floats of the record that `cdr_prepare` makes of one run and head."""
+    return int(_lib("channel_delta").tokb200_cdr_record(_i(dim), _i(vdim)))
+
+
+def cdr_records(n_rows: int, n_requests: int, heads: int, dim: int, vdim: int, device) -> torch.Tensor:
+    """Room for a step's records: every request's portion is cut into runs of four rows."""
+    return torch.empty((n_rows // CDR_RUN + n_requests, heads, cdr_record(dim, vdim)), dtype=torch.float32, device=device)
+
+
+def cdr_prepare(proj: torch.Tensor, qkv_at: int, b_at: int, pre: torch.Tensor, groups: int, heads: int, dim: int,
+                vdim: int, taps: int, conv_w, a_log, dt_bias, state: torch.Tensor, conv_off: int, q_start, state_slot,
+                records: torch.Tensor) -> None:
+    """Short convolution + silu of q, k, v (from `proj`'s columns qkv_at ..), unit vectors for q (times
+    dim^-1/2) and k, beta = sigmoid(proj[b_at ..]) and the decays exp(-exp(a_log) softplus(pre + dt_bias)), one a head and
+    key channel (`pre` float32, its first heads * dim columns), made into one record a run of four rows and
+    head (`cdr_records`).  The kept inputs in `state` are read, not moved on (`short_conv_state` does that)."""
+    channels, n = 2 * groups * dim + heads * vdim, proj.shape[0]
+    if proj.dtype != torch.float32 or pre.dtype != torch.float32 or pre.shape[0] != n or pre.shape[1] < heads * dim or \
+            state.dtype != torch.float32 or state.dim() != 2 or conv_w.numel() != channels * taps or \
+            conv_off + (taps - 1) * channels > state.shape[1] or max(qkv_at + channels, b_at + heads) > proj.shape[1] or \
+            a_log.numel() != heads or dt_bias.numel() != heads * dim or \
+            tuple(records.shape[1:]) != (heads, cdr_record(dim, vdim)) or \
+            records.shape[0] < n // CDR_RUN + q_start.shape[0] - 1:
+        raise ValueError("cdr_prepare: sizes of the products, the state, the taps or the records disagree")
+    _check(_lib("channel_delta").tokb200_cdr_prepare(
+        _sliced_ptr(proj), _i(_ld(proj)), _i(qkv_at), _i(b_at), _sliced_ptr(pre), _i(_ld(pre)), _i(groups), _i(heads), _i(dim),
+        _i(vdim), _i(taps), _ptr(conv_w), _ptr(a_log), _ptr(dt_bias), _ptr(state), _ll(state.shape[1]), _i(conv_off),
+        _ptr(q_start), _ptr(state_slot), _i(n), _i(q_start.shape[0] - 1), _ptr(records), _stream()), "cdr_prepare")
+
+
+def cdr_scan(records: torch.Tensor, heads: int, dim: int, vdim: int, state: torch.Tensor, q_start, state_slot,
+             o_out: torch.Tensor) -> None:
+    """The recurrence over every request's runs, head by head; `state` float32 [slots, n] holds the heads'
+    matrices transposed and padded ([heads, vdim, cdr_padded_dim(dim)]) at the start of a slot; `o_out` float32
+    [T, heads * vdim]."""
+    if state.dtype != torch.float32 or o_out.dtype != torch.float32 or o_out.shape[1] != heads * vdim or \
+            heads * vdim * cdr_padded_dim(dim) > state.shape[1] or tuple(records.shape[1:]) != (heads, cdr_record(dim, vdim)):
+        raise ValueError("cdr_scan: sizes of the state, the records or the output disagree")
+    _check(_lib("channel_delta").tokb200_cdr_scan(
+        _ptr(records), _i(heads), _i(dim), _i(vdim), _ptr(state), _ll(state.shape[1]), _ptr(q_start), _ptr(state_slot),
+        _i(q_start.shape[0] - 1), _ptr(o_out), _stream()), "cdr_scan")
+
+
+def cdr_step(proj: torch.Tensor, qkv_at: int, b_at: int, low_at: int, ra: int, rg: int, w2, pre, groups: int, heads: int,
+             dim: int, vdim: int, taps: int, conv_w, a_log, dt_bias, gain, eps: float, state: torch.Tensor, conv_off: int,
+             row_req, state_slot, shift: bool, out: torch.Tensor) -> None:
+    """A step in which every request brings ONE token: convolution, decay, recurrence, output norm and the sigmoid
+    gate in one kernel.  `pre` float32 [T, heads * (dim + vdim)]: the pre-activations of the decay and of the gate;
+    None: the kernel makes them from `proj`'s columns low_at .. + ra + rg and `w2` [heads * (dim + vdim), ra + rg].
+    `shift`: the kept inputs move on here (every head has q and k of its own); else `short_conv_state` follows."""
+    channels, n = 2 * groups * dim + heads * vdim, proj.shape[0]
+    if proj.dtype != torch.float32 or state.dtype != torch.float32 or state.dim() != 2 or tuple(out.shape) != (n, heads * vdim) or \
+            conv_w.numel() != channels * taps or conv_off + (taps - 1) * channels > state.shape[1] or gain.numel() != vdim or \
+            (shift and heads != groups) or a_log.numel() != heads or dt_bias.numel() != heads * dim:
+        raise ValueError("cdr_step: sizes of the state, the taps, the gain or the output disagree")
+    if (pre is None and (tuple(w2.shape) != (heads * (dim + vdim), ra + rg) or w2.dtype != out.dtype or
+                         low_at + ra + rg > proj.shape[1])) or \
+            (pre is not None and (pre.dtype != torch.float32 or tuple(pre.shape) != (n, heads * (dim + vdim)))):
+        raise ValueError("cdr_step: the second low-rank products or their weight have other sizes")
+    _check(_lib("channel_delta").tokb200_cdr_step(
+        _sliced_ptr(proj), _i(_ld(proj)), _i(qkv_at), _i(b_at), _i(low_at), _i(ra), _i(rg), _ptr(w2), _i(_tag(out)),
+        _ptr(pre), _i(groups), _i(heads), _i(dim), _i(vdim), _i(taps), _ptr(conv_w), _ptr(a_log), _ptr(dt_bias), _ptr(gain),
+        _f(eps), _ptr(state), _ll(state.shape[1]), _i(conv_off), _ptr(row_req), _ptr(state_slot), _i(n), _i(int(bool(shift))),
+        _ptr(out), _i(_tag(out)), _stream()), "cdr_step")
+
+
+def take_columns(proj: torch.Tensor, at: int, out: torch.Tensor) -> None:
+    """out [T, n] (dense) = columns at .. + n of the float32 product `proj`."""
+    n_rows, n = out.shape
+    if proj.dtype != torch.float32 or proj.shape[0] != n_rows or at + n > proj.shape[1]:
+        raise ValueError("take_columns: a float32 product that has the columns")
+    _check(_lib("channel_delta").tokb200_take_columns(
+        _sliced_ptr(proj), _i(_ld(proj)), _i(at), _i(n), _ptr(out), _i(_tag(out)), _i(n_rows), _stream()), "take_columns")
+
+
+# ---- a norm without statistics and the stream's steps around it ----
+def stream_update(x: torch.Tensor, y=None, base=None, carried=None, share=None, alpha=None, gain=None, bias=None,
+                  beside=None, out=None, rows=None) -> None:
+    """x <- (x or `base`, a float32 vector over the width) + y + share * carried, in place (each where given; x
+    float32 [T, H]; y [T, H] or float32 partial sums [S, T, H]; `carried` [T, H] with one float32 a row in `share`,
+    a column of a wider matrix).  With `out`: out = tanh(alpha x) * gain + bias of the new x, or x itself where `gain` is None; with
+    `beside` (float32 [T, H]) out is [T, 2 H] and its second half is `beside`.  `rows` (int32): only those rows of x
+    are read and x stays as it is."""
+    hidden = x.shape[-1]
+    n_rows = x.shape[0] if rows is None else rows.shape[0]
+    if x.dtype != torch.float32 or (gain is not None and (out is None or gain.dtype != torch.float32 or bias.dtype != torch.float32 or
+                                                          gain.numel() != hidden or bias.numel() != hidden)) or \
+            (out is not None and tuple(out.shape) != (n_rows, hidden * (2 if beside is not None else 1))) or \
+            (carried is not None and (tuple(carried.shape) != tuple(x.shape) or share.dtype != torch.float32 or
+                                      share.numel() != n_rows)) or \
+            (base is not None and (base.dtype != torch.float32 or base.numel() != hidden)) or \
+            (beside is not None and (beside.dtype != torch.float32 or beside.shape != x.shape)):
+        raise ValueError("stream_update: x is float32 [T, H]; vectors are float32 of H, matrices [T, H]")
+    n_partials, stride = _partials(y, x) if y is not None else (1, 0)
+    _check(_lib("dynamic_tanh").tokb200_stream_update(
+        _ptr(x), _ptr(y), _i(_tag(y) if y is not None else F32), _i(n_partials), _ll(stride), _ptr(base), _ptr(carried),
+        _i(_tag(carried) if carried is not None else F32), _sliced_ptr(share) if share is not None else _ptr(None),
+        _i(share.stride(0) if share is not None else 0), _i(int(gain is not None)), _f(alpha if alpha is not None else 0.0), _ptr(gain), _ptr(bias),
+        _ptr(beside), _ptr(out), _i(_tag(out) if out is not None else F32), _i(out.shape[1] if out is not None else 0),
+        _ptr(rows), _i(n_rows), _i(hidden), _stream()), "stream_update")
 
 
 # ---- queries, keys and values with unlike head sizes; routed experts ----
 def qkv_rotate_store(proj: torch.Tensor, at: int, bias, inv_freq, rot_dims: int, pos, slot, row_req, q_out, k_pool,
                      v_pool, heads: int, kv_heads: int, dim: int, vdim: int, row: int, q_gain=None, k_gain=None,
-                     eps: float = 0.0, temp=None, layout: str = "interleaved", head_norm_eps: Optional[float] = None) -> None:
+                     eps: float = 0.0, temp=None, layout: str = "interleaved", head_norm_eps: Optional[float] = None,
+                     magnitude: float = 1.0) -> None:
     """Bias, interleaved rotation of the first `rot_dims` lanes of every query and key head, and the
     cache write, from `proj`'s columns at .. (q, k, v); rows of `row` lanes a head, zero behind dim
     (queries, keys) and vdim (values).  `slot` None: no cache write.  `q_gain` / `k_gain` (float32, one a
@@ -1263,7 +1381,7 @@ def qkv_rotate_store(proj: torch.Tensor, at: int, bias, inv_freq, rot_dims: int,
     the head's queries.  `layout` "half": lane i of the rotated lanes pairs with lane i + rot_dims / 2 instead.
     `head_norm_eps` (a number): after the rotation every query and key head is divided by its own root mean
     square over its dim lanes, that eps inside the root.  `inv_freq` float64: the angle position * frequency is
-    taken in 64-bit and brought into one turn before its sine and cosine (float32: the 32-bit product).  `kv_heads` 0: `proj` holds queries only and nothing
+    taken in 64-bit and brought into one turn before its sine and cosine (float32: the 32-bit product).  `magnitude` multiplies cosine and sine (1 with `head_norm_eps`).  `kv_heads` 0: `proj` holds queries only and nothing
     but `q_out` is written (`slot`, `k_pool`, `v_pool` None)."""
     n = proj.shape[0]
     if layout not in ("interleaved", "half"):
@@ -1283,7 +1401,7 @@ def qkv_rotate_store(proj: torch.Tensor, at: int, bias, inv_freq, rot_dims: int,
         _ptr(inv_freq if wide else None), _i(rot_dims), _ptr(pos),
         _ptr(slot), _ptr(row_req), _ptr(q_out), _ptr(k_pool), _ptr(v_pool), _i(_tag(q_out)), _i(n), _i(heads),
         _i(kv_heads), _i(dim), _i(vdim), _i(row), _ptr(q_gain), _ptr(k_gain), _f(eps), _ptr(temp),
-        _i(int(layout == "half")), _i(int(head_norm_eps is not None)), _f(head_norm_eps or 0.0), _stream()),
+        _i(int(layout == "half")), _i(int(head_norm_eps is not None)), _f(head_norm_eps or 0.0), _f(magnitude), _stream()),
         "qkv_rotate_store")
 
 
@@ -1298,33 +1416,39 @@ def attention_gate(out: torch.Tensor, proj: torch.Tensor, at: int, heads: int, v
         _i(row), _stream()), "attention_gate")
 
 
-MOE_SCORES = {"softmax_of_chosen": 0, "sigmoid": 1}
+MOE_SCORES = {"softmax_of_chosen": 0, "sigmoid": 1, "softmax": 2}
 MOE_SHARED = {None: 0, "gated": 1, "one": 2}
 MOE_ACTIVATIONS = dict(ACTIVATIONS, clamped_swish=len(ACTIVATIONS))
 
 
 def moe_route(h: torch.Tensor, w: torch.Tensor, experts: int, top: int, shared, share: torch.Tensor,
               score: str = "softmax_of_chosen", correction: Optional[torch.Tensor] = None, groups: int = 1,
-              keep: int = 1, scale: float = 1.0) -> None:
+              keep: int = 1, scale: float = 1.0, identity: int = 0, group_worth: int = 2,
+              renormalize: bool = False) -> None:
     """Router logits z = w h in 32-bit (`w` float32 [experts (+ 1), hidden]; `h` float32 or bfloat16), then
     every expert's share of the token, zero where it is not chosen.  `score` "softmax_of_chosen": the `top`
     largest logits, share = softmax over them.  "sigmoid": s = sigmoid(z); the choice is made on s +
     `correction` (float32, one an expert, or None) among the experts of the `keep` best of `groups` equal
-    groups of neighbours (a group's worth: the sum of its two largest choice scores); share = s * `scale`.
+    groups of neighbours (a group's worth: the sum of its `group_worth` largest choice scores, 1 or 2); share =
+    s * `scale`, divided by the chosen scores' sum + 1e-20 where `renormalize` says so.  "softmax": the same with s
+    the softmax over all router outputs.  `identity` (not with "softmax_of_chosen"): that many router rows behind the
+    experts' stand for the token's input itself; they are chosen like experts (groups and correction run over both),
+    and the sum of their shares is one more column of `share`, the last.
     `shared`: None / False (no shared expert), "gated" / True (share[t, experts] = sigmoid of one more router
     row), "one" (share[t, experts] = 1)."""
     n, hidden = h.shape
     shared = {True: "gated", False: None}.get(shared, shared)
-    rows = experts + int(shared == "gated")
-    columns = experts + int(shared is not None)
+    rows = experts + identity + int(shared == "gated")
+    columns = experts + int(shared is not None) + int(identity > 0)
     if w.dtype != torch.float32 or tuple(w.shape) != (rows, hidden) or share.dtype != torch.float32 or \
             tuple(share.shape) != (n, columns):
         raise ValueError("moe_route: float32 router rows [experts (+ 1), hidden], shares float32 [T, experts (+ 1)]")
-    if correction is not None and (correction.dtype != torch.float32 or correction.numel() != experts):
+    if correction is not None and (correction.dtype != torch.float32 or correction.numel() != experts + identity):
         raise ValueError("moe_route: the correction is float32, one an expert")
     _check(_lib("moe").tokb200_moe_route(_ptr(h), _i(_tag(h)), _ptr(w), _i(hidden), _i(experts), _i(top),
                                          _i(MOE_SHARED[shared]), _ptr(share), _i(n), _i(MOE_SCORES[score]),
-                                         _ptr(correction), _i(groups), _i(keep), _f(scale), _stream()), "moe_route")
+                                         _ptr(correction), _i(groups), _i(keep), _f(scale), _i(identity), _i(group_worth),
+                                         _i(int(bool(renormalize))), _stream()), "moe_route")
 
 
 def moe_gate(gu: torch.Tensor, share: torch.Tensor, out: torch.Tensor, experts: int, ff: int, shared: bool,
@@ -1336,13 +1460,14 @@ def moe_gate(gu: torch.Tensor, share: torch.Tensor, out: torch.Tensor, experts: 
     g * sigmoid(alpha g) * (u + 1) (`shared_limit` for the shared expert's lanes).  `on_input`: the share
     multiplies the expert's input instead, out[t, c] = act(share * gate) * (share * up)."""
     n, inner = out.shape
-    if gu.shape[1] != 2 * inner or gu.dtype != out.dtype or tuple(share.shape) != (n, experts + int(shared)):
-        raise ValueError("moe_gate: input [T, 2 I], output [T, I] of one type, shares [T, experts (+ 1)]")
+    if gu.shape[1] != 2 * inner or gu.dtype != out.dtype or share.shape[0] != n or share.shape[1] < experts + int(shared):
+        raise ValueError("moe_gate: input [T, 2 I], output [T, I] of one type, shares [T, experts (+ 1) or more]")
     if activation not in MOE_ACTIVATIONS:
         raise ValueError(f"moe_gate: activation is one of {', '.join(MOE_ACTIVATIONS)}")
     _check(_lib("moe").tokb200_moe_gate(_ptr(gu), _ptr(share), _ptr(out), _i(_tag(gu)), _i(n), _i(inner), _i(experts),
                                         _i(ff), _i(int(shared)), _i(MOE_ACTIVATIONS[activation]), _f(limit),
-                                        _f(shared_limit), _f(alpha), _i(int(on_input)), _stream()), "moe_gate")
+                                        _f(shared_limit), _f(alpha), _i(int(on_input)), _i(share.shape[1]), _stream()),
+           "moe_gate")
 
 
 # ---- a short convolution across steps; a layer whose sublayers share one norm; learned positions ----

@@ -22,6 +22,8 @@ def all_variants():
         ("latent.cu", (), ()),
         ("layer_norm.cu", (), ()),
         ("delta_rule.cu", (), ()),
+        ("channel_delta.cu", (), ()),
+        ("dynamic_tanh.cu", (), ()),
         ("rotary_store.cu", (), ()),
         ("moe.cu", (), ()),
         ("short_conv.cu", (), ()),

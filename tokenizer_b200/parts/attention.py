@@ -140,6 +140,7 @@ class PagedAttention:
     graph_safe = True   # launches depend on device-side metadata only
     sink = None
     chunk = None        # n: keys are seen inside chunks of n positions counted from 0
+    keep_first = 0      # a sequence's first keys, seen whatever the window or the chunk says
     softcap = None      # c: a score s counts as c * tanh(s / c)
 
     def batch_annotations(self):
@@ -166,7 +167,8 @@ class PagedAttention:
                 ops.decode_attention_supported(self.nh, self.nkv, self.d):
             ops.decode_attention(
                 q, k_pool, v_pool, out, group.block_table, ctx.row_req, ctx.pos,
-                self.nh, self.nkv, self.d, group.page_size, self.window, self.scale, sink=sink, chunk=self.chunk, softcap=self.softcap)
+                self.nh, self.nkv, self.d, group.page_size, self.window, self.scale, sink=sink, chunk=self.chunk, softcap=self.softcap,
+                keep_first=self.keep_first)
             return
         wide, tiles = ctx.views.get(_WIDE_TILES.key), ctx.views.get(_TILES.key)
         singles = ctx.views.get(_SINGLES.key)
@@ -177,7 +179,8 @@ class PagedAttention:
             # (keys split over blocks, the group's heads as one tile), the portions to theirs
             ops.decode_attention(
                 q, k_pool, v_pool, out, group.block_table, ctx.row_req, ctx.pos,
-                self.nh, self.nkv, self.d, group.page_size, self.window, self.scale, rows=singles[0], sink=sink, chunk=self.chunk, softcap=self.softcap)
+                self.nh, self.nkv, self.d, group.page_size, self.window, self.scale, rows=singles[0], sink=sink, chunk=self.chunk, softcap=self.softcap,
+                keep_first=self.keep_first)
             wide, tiles = ctx.views[_LONG_WIDE_TILES.key], ctx.views[_LONG_TILES.key]
         if _PROMPT_KERNEL == "tcgen05" and q.dtype == torch.bfloat16 and \
                 wide is not None and ctx.max_q_len >= _WIDE_FROM and \
@@ -186,18 +189,21 @@ class PagedAttention:
             ops.attention_tcgen05(
                 q, k_pool, v_pool, out, group.block_table, ctx.row_req, ctx.pos,
                 wide[0], wide[1], self.nh, self.nkv, self.d, group.page_size,
-                self.window, self.scale, sink=sink, chunk=self.chunk, softcap=self.softcap)
+                self.window, self.scale, sink=sink, chunk=self.chunk, softcap=self.softcap,
+                keep_first=self.keep_first)
             return
         if q.dtype == torch.bfloat16 and tiles is not None and \
                 ops.prefill_attention_supported(self.nh, self.nkv, self.d):
             ops.prefill_attention(
                 q, k_pool, v_pool, out, group.block_table, ctx.row_req, ctx.pos,
                 tiles[0], tiles[1], self.nh, self.nkv, self.d, group.page_size,
-                self.window, self.scale, sink=sink, chunk=self.chunk, softcap=self.softcap)
+                self.window, self.scale, sink=sink, chunk=self.chunk, softcap=self.softcap,
+                keep_first=self.keep_first)
             return
         ops.paged_attention_generic(
             q, k_pool, v_pool, out, group.block_table, ctx.row_req, ctx.pos,
-            self.nh, self.nkv, self.d, group.page_size, self.window, self.scale, sink=sink, chunk=self.chunk, softcap=self.softcap)
+            self.nh, self.nkv, self.d, group.page_size, self.window, self.scale, sink=sink, chunk=self.chunk, softcap=self.softcap,
+                keep_first=self.keep_first)
 
 
 class GQAttention(PagedAttention):
@@ -381,7 +387,9 @@ class RotaryGQAttention(PagedAttention):
     with its `position` part (interleaved pairs or halves); `head_norm` (after the rotation every query and key
     head is divided by its root mean square over dim, `norm_eps` inside the root, no gain); `softcap` (a score s
     counts as softcap * tanh(s / softcap)); `output_gate` (the heads' outputs are multiplied by sigmoid(Wg h),
-    tensor `.g`, heads * vdim rows; the product rides in the stacked input product); `own_kv` False (the layer
+    tensor `.g`, heads * vdim rows; the product rides in the stacked input product); `unit_sink` (one added to
+    the softmax's denominator: a sink of score 0 for every head, no tensor); `keep_first` (the sequence's first
+    keys that every query sees although its window or chunk has passed them); `own_kv` False (the layer
     has no k and v tensors and is called on an earlier call's cache: it projects, rotates and norms queries
     only); `cache_chunk` (what the cache manager may give back, where other calls read this cache with chunks of
     their own: a chunk size that all of theirs divide, or None to keep every page)."""
@@ -419,6 +427,7 @@ class RotaryGQAttention(PagedAttention):
         self.dim, self.vdim = int(p["dim"]), int(p["vdim"])
         self.scale = float(p["scale"])
         self.window, self.chunk = p.get("window"), p.get("chunk")
+        self.keep_first = int(p.get("keep_first") or 0)
         self.softcap = float(p["softcap"]) if p.get("softcap") is not None else None
         self.own_kv = bool(p.get("own_kv", True))
         self.cache_chunk = p["cache_chunk"] if "cache_chunk" in p else self.chunk
@@ -457,6 +466,8 @@ class RotaryGQAttention(PagedAttention):
             self.temp = runtime.vector(store.get(x + ".temp"))
         if p.get("sink"):
             self.sink = runtime.vector(store.get(x + ".sink"))
+        elif p.get("unit_sink"):
+            self.sink = runtime.vector(torch.zeros(self.nh))
         w_o = store.get(x + ".o")
         if self.row != self.vdim:           # zero columns where the value lanes end
             wide = torch.zeros((self.hidden, self.nh, self.row), dtype=w_o.dtype)
@@ -471,7 +482,7 @@ class RotaryGQAttention(PagedAttention):
         return torch.cat(self._stack, dim=0), None
 
     def cache_need(self):
-        return CacheNeed(kv=KVNeed(self.nkv, self.row, self.window, chunk=self.cache_chunk))
+        return CacheNeed(kv=KVNeed(self.nkv, self.row, self.window, chunk=self.cache_chunk, keep_first=self.keep_first))
 
     def streamed_weights(self):
         return [self.out.weight] if self.inputs is None else [self.inputs.weight, self.out.weight]
@@ -489,6 +500,7 @@ class RotaryGQAttention(PagedAttention):
                              self.nkv if self.own_kv else 0, self.dim, self.vdim, self.row,
                              q_gain=self.q_gain, k_gain=self.k_gain, eps=self.norm_eps, temp=self.temp,
                              layout=getattr(self.position, "layout", "interleaved"),
+                             magnitude=getattr(self.position, "magnitude", 1.0),
                              head_norm_eps=self.norm_eps if self.head_norm else None)
         mixed = self.runtime.empty(ctx.n_tokens, self.nh * self.row)
         self.attend(q, mixed, ctx, group, cache)

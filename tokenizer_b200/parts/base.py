@@ -105,13 +105,16 @@ class KVNeed:
     that size which the mixer reads as both (`planes` = 1).  With a `window`, only the last
     window + 1 positions are ever read, and pages wholly before them are given back.  With a
     `chunk`, a query reads the keys of its own chunk of that many positions (counted from 0) only,
-    and pages wholly before the chunk of a request's next position are given back."""
+    and pages wholly before the chunk of a request's next position are given back.  The first
+    `keep_first` positions of a sequence stay readable whatever window and chunk say, and so do
+    their pages."""
 
     kv_heads: int
     head_dim: int
     window: Optional[int] = None
     planes: int = 2      # 2: keys and values; 1: one row a token that serves as both (a cached latent)
     chunk: Optional[int] = None
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)
@@ -255,6 +258,18 @@ class VectorScaledTerms:
     terms: List[Tuple[torch.Tensor, torch.Tensor]]
 
 
+@dataclass
+class StreamUpdate:
+    """What a sublayer (or what enters a pass) does to the stream: x <- (x or `base`) + y + share * carried.  y
+    [T, H] or float32 partial sums [S, T, H], or None; `base` float32 [H]: x starts anew from this vector;
+    `carried` [T, H] with one float32 a row in `share` (a sublayer's input that is handed through, weighed)."""
+
+    y: Optional[torch.Tensor] = None
+    base: Optional[torch.Tensor] = None
+    carried: Optional[torch.Tensor] = None
+    share: Optional[torch.Tensor] = None
+
+
 class ResidualStream:
     """The residual sum, kept in float32.  A part's output is not added at once:
     it stays pending until the next norm, which adds it while it reads the row
@@ -270,6 +285,7 @@ class ResidualStream:
         self._gated: Optional[GatedDelta] = None
         self._normed = None      # (terms, norm): a sublayer's output that is normed before it is added
         self._scaled: Optional[VectorScaledTerms] = None     # outputs still to be scaled by their vectors
+        self._update: Optional[StreamUpdate] = None          # an update of more than one addend
 
     @property
     def pending(self) -> Optional[torch.Tensor]:
@@ -279,6 +295,9 @@ class ResidualStream:
         if self._scaled is not None:
             scaled, self._scaled = self._scaled, None
             ops.scaled_add_norm(self.x, scaled.terms)      # in place as well
+        if self._update is not None:
+            update, self._update = self._update, None
+            ops.stream_update(self.x, update.y, update.base, update.carried, update.share)      # in place as well
         if self._gated is not None:
             g, self._gated = self._gated, None
             self._pending = torch.empty(self.x.shape, dtype=torch.float32, device=self.x.device)
@@ -287,7 +306,7 @@ class ResidualStream:
 
     @pending.setter
     def pending(self, value: Optional[torch.Tensor]) -> None:
-        self._pending, self._gated, self._normed, self._scaled = value, None, None, None
+        self._pending, self._gated, self._normed, self._scaled, self._update = value, None, None, None, None
 
     def add(self, delta) -> None:
         self.flush()
@@ -295,7 +314,24 @@ class ResidualStream:
             summed = torch.empty(self.x.shape, dtype=torch.float32, device=self.x.device)
             ops.scaled_sum(delta.terms, summed)
             delta = summed
+        if isinstance(delta, StreamUpdate):
+            self._update = delta
+            return
         self.pending = delta
+
+    def restart(self, update: StreamUpdate) -> None:
+        """The stream starts anew from `update` (which has a `base`); what was pending must have been taken."""
+        self.x = torch.empty_like(self.x)
+        self.pending = None
+        self._update = update
+
+    def take_update(self) -> StreamUpdate:
+        """What is pending, as one `StreamUpdate`, for a kernel that applies it on its way (empty: nothing)."""
+        if self._update is not None:
+            update, self._update = self._update, None
+            return update
+        y, self.pending = self.pending, None
+        return StreamUpdate(y)
 
     def add_normed(self, delta, post) -> None:
         """x += post(delta), with the norm `post` on the sublayer's OUTPUT: it stays pending, so
@@ -335,6 +371,9 @@ class ResidualStream:
         if self._scaled is not None and scaled is not None:
             terms, self._scaled = self._scaled, None
             return scaled(self.x, terms)
+        updating = getattr(norm, "forward_update", None)
+        if updating is not None and self._gated is None:
+            return updating(self.x, self.take_update())
         fused = getattr(norm, "forward_gated", None)
         if self._gated is not None and fused is not None and self.x.shape[0] <= self.GATED_NORM_ROWS:
             gated, self._gated = self._gated, None

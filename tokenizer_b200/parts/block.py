@@ -7,7 +7,7 @@ import torch
 
 from ..kernels import ops
 from ..weights.store import TensorSpec
-from .base import GatedDelta, register_part
+from .base import GatedDelta, StreamUpdate, register_part
 from .linear import Linear
 
 
@@ -57,7 +57,23 @@ class PreNormResidual:
             stream.add(self.feed_forward.forward(stream.normed(self.feed_forward_norm)))
 
 
+class PreNormMixerOnly:
+    """The same arrangement for a layer without a feed-forward: x += mixer(norm(x))."""
+
+    PARTS = {"mixer": "mixer", "mixer_norm": "norm"}
+
+    def __init__(self, mixer, mixer_norm):
+        self.mixer, self.mixer_norm = mixer, mixer_norm
+
+    def streamed_weights(self):
+        return list(getattr(self.mixer, "streamed_weights", lambda: [])())
+
+    def forward(self, stream, ctx, cache):
+        stream.add(self.mixer.forward(stream.normed(self.mixer_norm), ctx, cache))
+
+
 register_part("block", "pre_norm_residual", PreNormResidual)
+register_part("block", "pre_norm_mixer_only", PreNormMixerOnly)
 
 
 class ResidualGate:
@@ -189,6 +205,37 @@ class PassEntry:
         ops.stream_inject(stream.flush(), embedded if self.needs_embedding else None, self.vector)
 
 
+class PassProjection:
+    """What a pass of a looped stack of layers starts from: x <- W [x; x0] + row `index` of a tensor
+    [passes, hidden] (`tensor`), W (`projection`, [hidden, 2 hidden]) on the stream and, behind it, the embedding's
+    output.  What is pending on the stream is added while the product's operand is written; the product and the vector
+    stay pending in turn, so that the norm that follows adds them (the new stream is float32 whatever the
+    product's operands are)."""
+
+    needs_embedding = True
+
+    @staticmethod
+    def tensors(spec):
+        p = spec.params
+        return [TensorSpec(p["projection"], (p["hidden_size"], 2 * p["hidden_size"])),
+                TensorSpec(p["tensor"], (p["passes"], p["hidden_size"]))]
+
+    def __init__(self, spec, store, runtime):
+        p = spec.params
+        if not 0 <= int(p["index"]) < int(p["passes"]):
+            raise ValueError(f"pass {p['index']} of {p['passes']}")
+        self.runtime = runtime
+        self.proj = Linear(runtime.matrix(store.get(p["projection"])))
+        self.vector = runtime.vector(store.get(p["tensor"])[int(p["index"])])
+
+    def forward(self, stream, embedded):
+        update = stream.take_update()
+        joined = self.runtime.empty(stream.x.shape[0], 2 * stream.x.shape[1])
+        ops.stream_update(stream.x, update.y, update.base, update.carried, update.share, beside=embedded, out=joined)
+        stream.restart(StreamUpdate(self.proj.forward(joined, out_dtype=torch.float32, partials_ok=True), self.vector))
+
+
+register_part("injection", "pass_projection", PassProjection)
 register_part("block", "sandwich_norm_residual", SandwichNormResidual)
 register_part("block", "sandwich_norm_mixer_only", SandwichNormMixerOnly)
 register_part("injection", "pass_entry", PassEntry)

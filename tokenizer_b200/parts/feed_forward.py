@@ -11,7 +11,7 @@ import torch
 from ..config.spec import ConfigError
 from ..kernels import ops
 from ..weights.store import TensorSpec
-from .base import register_part
+from .base import StreamUpdate, register_part
 from .linear import Linear
 from .recurrent import SideProjection
 
@@ -179,17 +179,22 @@ class RoutedMLP:
     "clamped_swish" with `limit`, `shared_limit` and `alpha`: g = min(gate, limit), u = clamp(up, -limit,
     limit), g sigmoid(alpha g) (u + 1)); `share_on` ("output": an expert's output is multiplied by its weight;
     "input": its input is, expert(w h), which for products without biases is act(w gate) * (w up) on its inner
-    lanes and an unweighted sum behind the down product)."""
+    lanes and an unweighted sum behind the down product).  `score` "softmax": s = the softmax over all router
+    outputs, chosen as with "sigmoid"; `group_worth` (1 or 2): how many of a group's largest choice scores make up its
+    worth; `renormalize`: the chosen scores are divided by their sum.  `identity` n: the router has n more outputs
+    behind the experts', which stand for the layer's input itself and have no tensors: their shares' sum times the
+    input is left to whoever adds the output to the stream (`StreamUpdate`)."""
 
     @staticmethod
     def tensors(spec):
         p, x = spec.params, spec.prefix
         hidden, inner = p["hidden_size"], p["expert_inner"]
+        outputs = p["experts"] + int(p.get("identity") or 0)
         out = []
         for e in range(p["experts"]):
             out += [TensorSpec(f"{x}.e{e}.gate", (inner, hidden)), TensorSpec(f"{x}.e{e}.up", (inner, hidden)),
                     TensorSpec(f"{x}.e{e}.down", (hidden, inner))]
-        out.append(TensorSpec(x + ".router", (p["experts"], hidden)))
+        out.append(TensorSpec(x + ".router", (outputs, hidden)))
         if p.get("shared_inner"):
             s = p["shared_inner"]
             out += [TensorSpec(x + ".shared.gate", (s, hidden)), TensorSpec(x + ".shared.up", (s, hidden)),
@@ -197,7 +202,7 @@ class RoutedMLP:
             if p.get("shared_gate", True):
                 out.append(TensorSpec(x + ".shared.sg", (1, hidden)))
         if p.get("correction"):
-            out.append(TensorSpec(x + ".correction", (p["experts"],), "normal", 0.1))
+            out.append(TensorSpec(x + ".correction", (outputs,), "normal", 0.1))
         return out
 
     def __init__(self, spec, store, runtime):
@@ -209,8 +214,10 @@ class RoutedMLP:
         if self.activation not in ops.MOE_ACTIVATIONS:
             raise ConfigError(f"routed feed-forward knows the activations {', '.join(ops.MOE_ACTIVATIONS)}; "
                               f"found {self.activation}")
-        if not 1 <= self.top <= self.experts or self.experts > 1024:
-            raise ConfigError(f"a token uses 1 .. experts of at most 1024 experts; found top {self.top} of {self.experts}")
+        self.identity = int(p.get("identity") or 0)
+        outputs = self.experts + self.identity
+        if not 1 <= self.top <= outputs or outputs > 1024:
+            raise ConfigError(f"a token uses 1 .. experts of at most 1024 experts; found top {self.top} of {outputs}")
         self.score = p.get("score", "softmax_of_chosen")
         self.groups, self.group_keep = int(p.get("groups", 1)), int(p.get("group_keep", 1))
         self.route_scale = float(p.get("route_scale", 1.0))
@@ -221,9 +228,12 @@ class RoutedMLP:
             raise ConfigError(f"an expert's weight multiplies its output or its input; found {self.share_on}")
         if self.score not in ops.MOE_SCORES:
             raise ConfigError(f"a router scores by one of {', '.join(ops.MOE_SCORES)}; found {self.score}")
-        if self.groups < 1 or self.experts % self.groups or not 1 <= self.group_keep <= self.groups or \
-                self.group_keep * (self.experts // self.groups) < self.top:
-            raise ConfigError(f"{self.experts} experts in {self.groups} equal groups of which {self.group_keep} are kept "
+        self.group_worth, self.renormalize = int(p.get("group_worth", 2)), bool(p.get("renormalize"))
+        if self.identity and self.score == "softmax_of_chosen":
+            raise ConfigError("identity experts need a router that scores by sigmoid or by the softmax over all its outputs")
+        if self.groups < 1 or outputs % self.groups or not 1 <= self.group_keep <= self.groups or \
+                self.group_keep * (outputs // self.groups) < self.top:
+            raise ConfigError(f"{outputs} experts in {self.groups} equal groups of which {self.group_keep} are kept "
                               f"cannot give a token {self.top} experts")
         self.shared_mode = None if not self.shared else "gated" if p.get("shared_gate", True) else "one"
         self.correction = runtime.vector(store.get(x + ".correction")) if p.get("correction") else None
@@ -241,14 +251,17 @@ class RoutedMLP:
 
     def forward(self, h):
         n = h.shape[0]
-        share = torch.empty((n, self.experts + (1 if self.shared else 0)), dtype=torch.float32, device=h.device)
+        columns = self.experts + (1 if self.shared else 0) + (1 if self.identity else 0)
+        share = torch.empty((n, columns), dtype=torch.float32, device=h.device)
         ops.moe_route(h, self.router, self.experts, self.top, self.shared_mode, share, score=self.score,
-                      correction=self.correction, groups=self.groups, keep=self.group_keep, scale=self.route_scale)
+                      correction=self.correction, groups=self.groups, keep=self.group_keep, scale=self.route_scale,
+                      identity=self.identity, group_worth=self.group_worth, renormalize=self.renormalize)
         act = self.runtime.empty(n, self.inner)
         ops.moe_gate(self.gate_up.forward(h), share, act, self.experts, self.ff, bool(self.shared), self.activation,
                      limit=self.limit, shared_limit=self.shared_limit, alpha=self.alpha,
                      on_input=self.share_on == "input")
-        return self.down.forward(act, partials_ok=True)
+        out = self.down.forward(act, partials_ok=True)
+        return StreamUpdate(out, carried=h, share=share[:, columns - 1]) if self.identity else out
 
 
 register_part("feed_forward", "gated_mlp", GatedMLP)

@@ -1,5 +1,6 @@
 """RMSNorm: y = x / sqrt(mean(x^2) + eps) * gain, statistics in float32
-(reference: qwen-infer/src/model.rs:594-599, 616, 749); and the layer norm with gain and bias."""
+(reference: qwen-infer/src/model.rs:594-599, 616, 749); the layer norm with gain and bias; and the norm
+without statistics, tanh(alpha x) * gain + bias."""
 from __future__ import annotations
 
 import torch
@@ -129,5 +130,44 @@ class LayerNorm:
         return out
 
 
+class DynamicTanh:
+    """tanh(alpha x) * gain + bias, element by element: no mean, no variance.  Tensors: the gain under the norm's
+    name, `.b` (the bias) and `.alpha` (one number, shape []).  `scale` (optional): a constant that gain and
+    bias are multiplied by in float32, for a model whose logits are the head's product times a constant (the final
+    norm carries it).  It takes a pending update of the stream into its own kernel (`csrc/dynamic_tanh.cu`)."""
+
+    @staticmethod
+    def tensors(spec):
+        name = tensor_name(spec)
+        return [TensorSpec(name, (spec.params["size"],), "one_plus_normal"),
+                TensorSpec(name + ".b", (spec.params["size"],), "normal"),
+                TensorSpec(name + ".alpha", (), "one_plus_normal", 0.1)]
+
+    def __init__(self, spec, store, runtime):
+        self.size = int(spec.params["size"])
+        self.runtime = runtime
+        name = tensor_name(spec)
+        scale = float(spec.params.get("scale", 1.0))
+        self.alpha = float(store.get(name + ".alpha").to(torch.float32))
+        self.gain = (runtime.vector(store.get(name)) * scale).contiguous()
+        self.bias = (runtime.vector(store.get(name + ".b")) * scale).contiguous()
+
+    def forward_update(self, x, update):
+        """The pending update is applied to x in place, then the norm of the new x: one kernel."""
+        out = self.runtime.empty(x.shape[0], self.size)
+        ops.stream_update(x, update.y, update.base, update.carried, update.share, alpha=self.alpha, gain=self.gain,
+                          bias=self.bias, out=out)
+        return out
+
+    def forward(self, x, delta=None, rows=None):
+        if rows is not None and delta is not None:
+            ops.residual_add(x, delta)
+            delta = None
+        out = self.runtime.empty(x.shape[0] if rows is None else rows.shape[0], self.size)
+        ops.stream_update(x, delta, alpha=self.alpha, gain=self.gain, bias=self.bias, out=out, rows=rows)
+        return out
+
+
+register_part("norm", "dynamic_tanh", DynamicTanh)
 register_part("norm", "rms_norm", RMSNorm)
 register_part("norm", "layer_norm", LayerNorm)

@@ -1,4 +1,5 @@
-"""Recurrent mixers: minGRU and the gated delta rule (`GatedDeltaNet`, below).
+"""Recurrent mixers: minGRU, the gated delta rule (`GatedDeltaNet`, below), the delta rule with a decay a
+key channel (`ChannelDeltaNet`) and the state-space recurrence (`Mamba2`).
 
 minGRU: a gated recurrence whose gates read only the current token.
 
@@ -17,7 +18,7 @@ import torch
 
 from ..config.spec import ConfigError
 from ..kernels import ops
-from ..weights.store import TensorSpec
+from ..weights.store import FreeSize, TensorSpec
 from .base import CacheNeed, StateNeed, register_part
 from .linear import Linear
 
@@ -108,7 +109,7 @@ def stacked_rows(weights, multiple: int = 8):
     rows = sum(w.shape[0] for w in weights)
     spare = -rows % multiple
     if spare:
-        weights = list(weights) + [torch.zeros((spare, weights[0].shape[1]), dtype=weights[0].dtype)]
+        weights = list(weights) + [torch.zeros((spare, weights[0].shape[1]), dtype=weights[0].dtype, device=weights[0].device)]
     return torch.cat(weights, dim=0)
 
 
@@ -215,6 +216,121 @@ class GatedDeltaNet:
         return self.forward_projected(self.inputs.forward(h, out_dtype=torch.float32), 0, ctx, cache)
 
 
+# A decoding step of up to this many rows makes the decay's and the gate's second low-rank products inside the
+# step's kernel (every block reads its head's rows of the weight); more rows share one product in front of it
+CHANNEL_STEP_ROWS = 16
+
+
+class ChannelDeltaNet:
+    """The delta rule with one decay a key channel: per head a matrix state S (dim x vdim, float32), row c of
+    which every token multiplies by its own decay g[c]:
+        S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q.
+    q, k, v and beta as in `GatedDeltaNet` (value head i uses q/k head i // (heads / kv_heads)); the decays
+    are g = exp(-exp(A_log) softplus(W_a2 (W_a1 h) + dt_bias)), heads x dim of them, through a bottleneck (`.a1`
+    [rank, hidden], `.a2` [heads * dim, rank]; the file says the rank); every head's o is divided by its root mean square
+    over vdim, scaled by the gain `norm` and by sigmoid(W_g2 (W_g1 h)) (`.g1`, `.g2`, a bottleneck of its own); then Wo.
+    The input product (q, k, v, beta and both bottlenecks, stacked) is written in float32; everything behind it
+    but the second products' operands is 32-bit (`csrc/channel_delta.cu`).
+
+    Per request it keeps, in one state slot: the heads' matrices and the convolution's last taps - 1 inputs."""
+
+    graph_safe = True    # launches depend on device-side metadata alone
+
+    @staticmethod
+    def tensors(spec):
+        p, x = spec.params, spec.prefix
+        hidden, heads, groups, dim, vdim, taps = (p["hidden_size"], p["heads"], p["kv_heads"], p["dim"], p["vdim"],
+                                                  p["conv"])
+        decay_rank, gate_rank = FreeSize(x + ".a1", dim), FreeSize(x + ".g1", vdim)
+        return [TensorSpec(x + ".q", (groups * dim, hidden)), TensorSpec(x + ".q.conv", (groups * dim, taps), "normal", 0.5),
+                TensorSpec(x + ".k", (groups * dim, hidden)), TensorSpec(x + ".k.conv", (groups * dim, taps), "normal", 0.5),
+                TensorSpec(x + ".v", (heads * vdim, hidden)), TensorSpec(x + ".v.conv", (heads * vdim, taps), "normal", 0.5),
+                TensorSpec(x + ".b", (heads, hidden)), TensorSpec(x + ".A_log", (heads,), "normal", 0.5),
+                TensorSpec(x + ".norm", (vdim,), "one_plus_normal"),
+                TensorSpec(x + ".a1", (decay_rank, hidden)), TensorSpec(x + ".a2", (heads * dim, decay_rank), "normal", 0.1),
+                TensorSpec(x + ".dt_bias", (heads * dim,), "normal", 0.5),
+                TensorSpec(x + ".g1", (gate_rank, hidden)), TensorSpec(x + ".g2", (heads * vdim, gate_rank), "normal", 0.1),
+                TensorSpec(x + ".o", (hidden, heads * vdim))]
+
+    def __init__(self, spec, store, runtime):
+        p, x = spec.params, spec.prefix
+        self.runtime = runtime
+        self.hidden = int(p["hidden_size"])
+        self.heads, self.groups = int(p["heads"]), int(p["kv_heads"])
+        self.dim, self.vdim, self.taps = int(p["dim"]), int(p["vdim"]), int(p["conv"])
+        self.eps = float(p["eps"])
+        if self.groups <= 0 or self.heads % self.groups:
+            raise ConfigError(f"{self.heads} value heads do not divide into {self.groups} query/key heads")
+        self.dim_padded = ops.cdr_padded_dim(self.dim)
+        if not self.dim_padded or not 1 <= self.taps <= 16:
+            raise ConfigError(f"the delta rule by channels takes heads of up to 512 lanes and convolutions of up to 16 "
+                              f"taps; found {self.dim} and {self.taps}")
+        self.channels = 2 * self.groups * self.dim + self.heads * self.vdim
+        # the bottlenecks' ranks in whole 8s: zero rows of the first product meet zero columns of the second
+        a1, g1 = stacked_rows([store.get(x + ".a1")]), stacked_rows([store.get(x + ".g1")])
+        a2, g2 = store.get(x + ".a2"), store.get(x + ".g2")
+        self.ra, self.rg = a1.shape[0], g1.shape[0]
+        second = torch.zeros((self.heads * (self.dim + self.vdim), self.ra + self.rg), dtype=a2.dtype, device=a2.device)
+        second[:self.heads * self.dim, :a2.shape[1]] = a2
+        second[self.heads * self.dim:, self.ra:self.ra + g2.shape[1]] = g2
+        self.second = Linear(runtime.matrix(second))       # both second products as one, block by block
+        # the stacked input product: q, k, v | the bottlenecks | beta
+        self.low_at = self.channels
+        self.b_at = self.channels + self.ra + self.rg
+        self.inputs = Linear(runtime.matrix(stacked_rows([store.get(x + ".q"), store.get(x + ".k"), store.get(x + ".v"),
+                                                          a1, g1, store.get(x + ".b")])))
+        self.conv_w = runtime.vector(torch.cat([store.get(x + f".{n}.conv").to(torch.float32) for n in "qkv"], dim=0))
+        self.a_log = runtime.vector(store.get(x + ".A_log"))
+        self.dt_bias = runtime.vector(store.get(x + ".dt_bias"))
+        self.gain = runtime.vector(store.get(x + ".norm"))
+        self.out = Linear(runtime.matrix(store.get(x + ".o")))
+        # a slot: [heads, vdim, dim_padded] and behind it [taps - 1, channels], in whole 4s of floats
+        self.conv_off = self.heads * self.vdim * self.dim_padded
+        self.state_floats = -(-(self.conv_off + (self.taps - 1) * self.channels) // 4) * 4
+
+    def shape_key(self, q_lens):
+        return "channel_delta1" if max(q_lens) == 1 else "channel_delta"      # the kernels' choice
+
+    def cache_need(self):
+        return CacheNeed(state=StateNeed((self.state_floats,)))
+
+    def streamed_weights(self):
+        return [self.inputs.weight, self.second.weight, self.out.weight]
+
+    def _second_products(self, proj):
+        """The decay's and the gate's pre-activations, float32 [T, heads * (dim + vdim)]."""
+        low = self.runtime.empty(proj.shape[0], self.ra + self.rg)
+        ops.take_columns(proj, self.low_at, low)
+        return self.second.forward(low, out_dtype=torch.float32)
+
+    def forward(self, h, ctx, cache):
+        n, heads = ctx.n_tokens, self.heads
+        proj = self.inputs.forward(h, out_dtype=torch.float32)
+        y = self.runtime.empty(n, heads * self.vdim)
+        if ctx.max_q_len == 1 and _ONE_KERNEL_STEP:
+            # every request brings one token: one kernel behind the input product (a decoding step is bound by
+            # its launches)
+            shift = heads == self.groups
+            pre = self._second_products(proj) if n > CHANNEL_STEP_ROWS else None
+            ops.cdr_step(proj, 0, self.b_at, self.low_at, self.ra, self.rg, self.second.weight, pre, self.groups, heads,
+                         self.dim, self.vdim, self.taps, self.conv_w, self.a_log, self.dt_bias, self.gain, self.eps,
+                         cache.state, self.conv_off, ctx.row_req, ctx.state_slot, shift, y)
+            if not shift:
+                ops.short_conv_state(proj, 0, self.channels, self.taps, cache.state, self.conv_off, ctx.q_start,
+                                     ctx.state_slot)
+            return self.out.forward(y, partials_ok=True)
+        pre = self._second_products(proj)
+        records = ops.cdr_records(n, ctx.q_start.shape[0] - 1, heads, self.dim, self.vdim, proj.device)
+        ops.cdr_prepare(proj, 0, self.b_at, pre, self.groups, heads, self.dim, self.vdim, self.taps, self.conv_w, self.a_log,
+                        self.dt_bias, cache.state, self.conv_off, ctx.q_start, ctx.state_slot, records)
+        ops.short_conv_state(proj, 0, self.channels, self.taps, cache.state, self.conv_off, ctx.q_start, ctx.state_slot)
+        o = torch.empty((n, heads * self.vdim), dtype=torch.float32, device=proj.device)
+        ops.cdr_scan(records, heads, self.dim, self.vdim, cache.state, ctx.q_start, ctx.state_slot, o)
+        ops.gdn_out_norm(o, pre, heads * self.dim, self.gain, 1.0, self.eps, y, heads, self.vdim, ctx.row_req,
+                         gate_kind="sigmoid")
+        return self.out.forward(y, partials_ok=True)
+
+
 class Mamba2:
     """The selective state-space mixer with a scalar decay a head (Mamba-2).  With inner = heads * vdim,
     N = `state` lanes and G = `groups`: the input product W_in h is [z: inner | x: inner | B: G N | C: G N |
@@ -301,3 +417,4 @@ class Mamba2:
 register_part("mixer", "mamba2", Mamba2)
 register_part("mixer", "min_gru", MinGRU)
 register_part("mixer", "gated_delta_net", GatedDeltaNet)
+register_part("mixer", "channel_delta_net", ChannelDeltaNet)

@@ -13,20 +13,26 @@ from typing import Dict, Optional
 import torch
 
 from .safetensors_io import write_safetensors
+from .store import FreeSize
+
+
+def sized(shape, sizes: Optional[Dict[str, int]] = None):
+    """The shape as plain numbers; a dimension that the file decides takes `sizes[name]`, else its default."""
+    return tuple((sizes or {}).get(d.name, int(d)) if isinstance(d, FreeSize) else int(d) for d in shape)
 
 
 def random_tensors(specs, seed: int, scale: Optional[Dict[str, float]] = None,
-                   dtype: torch.dtype = torch.bfloat16) -> Dict[str, torch.Tensor]:
-    """`scale` maps a regular expression over tensor names to a factor applied
+                   dtype: torch.dtype = torch.bfloat16, sizes: Optional[Dict[str, int]] = None) -> Dict[str, torch.Tensor]:
+    """`sizes`: what the dimensions that a file decides (`FreeSize`) are to be, by name.  `scale` maps a regular expression over tensor names to a factor applied
     to the drawn values (tests sharpen attention by scaling q and k)."""
     generator = torch.Generator(device="cpu")
     generator.manual_seed(int(seed))
     tensors = {}
     for spec in sorted(specs, key=lambda s: s.name):
         if spec.init == "zeros":
-            value = torch.zeros(spec.shape, dtype=torch.float32)
+            value = torch.zeros(sized(spec.shape, sizes), dtype=torch.float32)
         else:
-            value = torch.randn(spec.shape, generator=generator, dtype=torch.float32) * spec.std
+            value = torch.randn(sized(spec.shape, sizes), generator=generator, dtype=torch.float32) * spec.std
             if spec.init == "one_plus_normal":
                 value = value + 1.0
             elif spec.init != "normal":
@@ -60,16 +66,16 @@ class SeededTensors:
         return len(self.specs)
 
     def shape_of(self, name: str):
-        return tuple(self.specs[name].shape)
+        return sized(self.specs[name].shape)
 
     def __getitem__(self, name: str) -> torch.Tensor:
         import zlib
         spec = self.specs[name]
         if spec.init == "zeros":
-            return torch.zeros(spec.shape, dtype=self.dtype, device=self.device)
+            return torch.zeros(sized(spec.shape), dtype=self.dtype, device=self.device)
         generator = torch.Generator(device=self.device)
         generator.manual_seed((self.seed * 1000003 + zlib.crc32(name.encode())) & 0x7FFFFFFFFFFFFFFF)
-        value = torch.randn(spec.shape, generator=generator, dtype=torch.float32, device=self.device) * spec.std
+        value = torch.randn(sized(spec.shape), generator=generator, dtype=torch.float32, device=self.device) * spec.std
         if spec.init == "one_plus_normal":
             value = value + 1.0
         elif spec.init != "normal":
@@ -79,7 +85,7 @@ class SeededTensors:
 
 def write_random_model(folder: str, config, seed: int,
                        scale: Optional[Dict[str, float]] = None,
-                       dtype: torch.dtype = torch.bfloat16) -> str:
+                       dtype: torch.dtype = torch.bfloat16, sizes: Optional[Dict[str, int]] = None) -> str:
     """Create `folder` with config.json and model.safetensors for `config`
     (a registered typed configuration)."""
     from ..parts.model import declared_tensors  # parts declare what they need
@@ -87,7 +93,7 @@ def write_random_model(folder: str, config, seed: int,
     os.makedirs(folder, exist_ok=True)
     specs = declared_tensors(config.model_spec())
     write_safetensors(os.path.join(folder, "model.safetensors"),
-                      random_tensors(specs, seed, scale, dtype))
+                      random_tensors(specs, seed, scale, dtype, sizes))
     with open(os.path.join(folder, "config.json"), "w") as fh:
         json.dump(config.to_dict(), fh, indent=1)
     return folder

@@ -19,9 +19,19 @@ import torch
 from .safetensors_io import WeightError, read_safetensors
 
 
+class FreeSize(int):
+    """A dimension that the weight file decides, not the configuration (the rank of a bottleneck): any size of
+    at least one fits, the same one wherever `name` stands.  Random-weights mode draws `default`."""
+
+    def __new__(cls, name: str, default: int):
+        value = super().__new__(cls, default)
+        value.name = name
+        return value
+
+
 @dataclass(frozen=True)
 class TensorSpec:
-    """`init` tells random-weights mode what to draw: "normal" (mean 0),
+    """A dimension of `shape` may be a `FreeSize`.  `init` tells random-weights mode what to draw: "normal" (mean 0),
     "one_plus_normal" (norm gains), "zeros"; `std` is its scale."""
 
     name: str
@@ -84,10 +94,11 @@ class WeightStore:
         missing = sorted(name for name in wanted if name not in self.tensors)
         unexpected = sorted(
             name for name in self.tensors if name not in wanted and name not in ignorable)
+        free: Dict[str, int] = {}
         wrong = sorted(
             (name, self._shape(name), shape)
             for name, shape in wanted.items()
-            if name in self.tensors and self._shape(name) != shape)
+            if name in self.tensors and not self._fits(self._shape(name), shape, free))
         if not (missing or unexpected or wrong):
             return
         lines = [f"{self.source} does not fit the model:"]
@@ -98,6 +109,14 @@ class WeightStore:
         for name, found, shape in wrong:
             lines.append(f"  wrong shape: {name} is {list(found)}, the model needs {list(shape)}")
         raise WeightError("\n".join(lines))
+
+    @staticmethod
+    def _fits(found: Tuple[int, ...], wanted: Tuple[int, ...], free: Dict[str, int]) -> bool:
+        """Whether a stored shape is the declared one; `free` remembers the sizes that the file has decided."""
+        if len(found) != len(wanted):
+            return False
+        return all(have >= 1 and free.setdefault(want.name, have) == have if isinstance(want, FreeSize) else have == want
+                   for have, want in zip(found, wanted))
 
     def _shape(self, name: str) -> Tuple[int, ...]:
         """A tensor's shape; a source that makes tensors on demand tells it without making one."""
