@@ -3,7 +3,7 @@
 weights on one B200.  Prints ONE JSON line.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--impl ours|reference]
-                    [--config 0.5b|1.5b-mixed|7b|pufuzen|katopel|vizonex|zobelorn]
+                    [--config 0.5b|1.5b-mixed|7b|pufuzen|katopel|vizonex|zobelorn|kazepel]
 
 A "step" is one decode step of the whole batch.  `value` is decoded tokens a
 second timed on the device over K steps that never return to the host
@@ -196,13 +196,15 @@ def main():
     parser.add_argument("--batch", type=int, default=8)
     parser.add_argument("--layers", type=int, default=SIZES["num_hidden_layers"])
     parser.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    parser.add_argument("--config", default="0.5b", choices=["0.5b", "1.5b-mixed", "7b", "pufuzen", "katopel", "vizonex", "zobelorn"],
+    parser.add_argument("--config", default="0.5b", choices=["0.5b", "1.5b-mixed", "7b", "pufuzen", "katopel", "vizonex", "zobelorn",
+                                                           "kazepel"],
                         help="0.5b: the headline line; 7b: the same at Qwen2.5-7B sizes with 8,192-token "
                              "contexts; 1.5b-mixed: 32 requests through the scheduler at Qwen2.5-1.5B sizes; "
                              "pufuzen: prefill and decoding of the Pufuzen design at two widths beside Qwen2 at "
                              "equal width, depth and parameters, and its kernels alone; katopel: the same for the Katopel design; "
                              "vizonex: the Vizonex design beside the Katopel design at equal width, depth and parameters; "
-                             "zobelorn: the Zobelorn design beside Qwen2 at equal width, depth, heads and parameters")
+                             "zobelorn: the Zobelorn design beside Qwen2 at equal width, depth, heads and parameters; "
+                             "kazepel: the Kazepel design beside the Katopel design at equal width, depth and parameters")
     parser.add_argument("--context", type=int, default=8192, help="--config 7b: tokens held before decoding")
     parser.add_argument("--layer-phases", action="store_true",
                         help="print where the time of the whole-layer kernel (TOKB200_LAYER=fused) goes, phase by "
@@ -217,7 +219,7 @@ def main():
     parser.add_argument("--only-decode", action="store_true",
                         help="time the decode steps only and print a short line (for profiling)")
     parser.add_argument("--only-kernels", action="store_true",
-                        help="--config katopel, vizonex, zobelorn: the kernels alone, without the models")
+                        help="--config katopel, vizonex, zobelorn, kazepel: the kernels alone, without the models")
     parser.add_argument("--only-prefill", action="store_true",
                         help="time the 2,048-token prefill only and print a short line (for profiling)")
     args = parser.parse_args()
@@ -247,6 +249,8 @@ def main():
         return run_vizonex(args)
     if args.config == "zobelorn":
         return run_zobelorn(args)
+    if args.config == "kazepel":
+        return run_kazepel(args)
     args.steps = max(1, min(args.steps, NEW_TOKENS - args.warmup - 1))
 
     import torch
@@ -1523,6 +1527,258 @@ def run_zobelorn(args):
         "unit": "tokens/s", "n_gpus": 1, "steps": steps, "warmup": args.warmup, "dtype": "bf16",
         "data": "synthetic: random weights drawn on the device, uniform random token ids",
         "config": {"sizes": ZOBELORN_SIZES, "prefill_tokens": PREFILL_TOKENS, "decode_context": context,
+                   "peaks": pk["source"], "hbm_gbs": pk["hbm_gbs"],
+                   "l2": "kernels alone: inputs larger than L2 and a 256 MB write between timed launches"},
+        "models": models, "kernels": kernels}))
+    return 0
+
+
+# ---- the Kazepel design beside the Katopel design at equal width, depth and parameter count ----
+KAZEPEL_SIZES = {
+    # width; attention of `heads` over `kv_heads` heads of dim / vdim lanes (a window of `window` keys with the first
+    # `keep` tokens kept, `rot` rotated lanes under yarn's scaling); the delta rule with a decay a key channel (heads over
+    # kv heads, dim x vdim matrices, taps; its bottlenecks have the rank of a head); `experts` experts and `identity`
+    # identity experts in `groups` groups of which `keep_groups` are kept, of which a token uses `top`.  The
+    # experts' width is chosen so that the model has the parameters of the Katopel model of the same name.
+    "1k": dict(width=1024, heads=16, kv_heads=4, dim=64, vdim=64, window=1024, keep=16, rot=32, d_heads=8, d_kv=8, d_dim=128,
+               d_vdim=128, taps=4, experts=8, identity=4, groups=4, keep_groups=2, top=2, vocab=32000, layers=8),
+    "2k": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, window=1024, keep=16, rot=64, d_heads=16, d_kv=16,
+               d_dim=128, d_vdim=128, taps=4, experts=8, identity=4, groups=4, keep_groups=2, top=2, vocab=32000, layers=8),
+}
+
+
+def kazepel_config(z, ff, loop=None):
+    """Delta rule and attention in turn, every layer with experts; no loop unless asked for, so that every layer has
+    weights of its own as in the model beside it."""
+    import tokenizer_b200 as tb
+    moe = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0},
+           "router": {"experts": z["experts"], "top": z["top"], "identity": z["identity"],
+                      "groups": {"count": z["groups"], "keep": z["keep_groups"]}}}
+    delta = {"heads": z["d_heads"], "kv_heads": z["d_kv"], "dim": z["d_dim"], "vdim": z["d_vdim"], "conv": z["taps"]}
+    attn = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5,
+            "mask": {"size": z["window"], "keep_first": z["keep"]},
+            "rot": {"base": 500000.0, "dims": z["rot"], "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    layers = [{"type": "channel_delta", "mixer": delta, "mlp": moe}, {"type": "attention", "mixer": attn, "mlp": moe}]
+    raw = {"architecture": "Kazepel", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+           "layers": [layers[i % 2] for i in range(z["layers"])]}
+    if loop is not None:
+        raw["loop"] = dict(zip(("start", "stop", "times"), loop))
+    return tb.config.KazepelConfig.from_dict(raw)
+
+
+def run_kazepel(args):
+    """Prefill (one step of 2,048 tokens) and decoding (batch 1 and `--batch`, 2,048-token contexts) of the Kazepel
+    design at two widths, beside the closest design that was there, Katopel (the delta rule with one decay a head,
+    attention inside chunks, routed experts), at the same width and depth with the experts' width that gives both the
+    same parameters, and once more with four of its layers looped twice; then the design's own kernels alone beside the
+    like kernels of the other paths, each on inputs larger than L2, against the measured copy peak."""
+    import numpy as np
+    import torch
+    from tokenizer_b200.kernels import ops
+    from tokenizer_b200.parts.attention import RowTiles
+    from tokenizer_b200.parts.linear import Linear
+    from tokenizer_b200.parts.model import declared_tensors
+
+    torch.cuda.set_device(0)
+    pk = peaks()
+    gen = torch.Generator().manual_seed(99)
+    context, steps = 2048, max(8, min(args.steps, 64))
+    timed = device_timed
+    count = lambda config: sum(int(torch.tensor(t.shape).prod()) for t in declared_tensors(config.model_spec()))
+
+    models = {}
+    for name, z in KAZEPEL_SIZES.items():
+        if args.only_kernels:
+            break
+        beside = katopel_config(KATOPEL_SIZES[name])
+        base, step = count(kazepel_config(z, 64)), count(kazepel_config(z, 128)) - count(kazepel_config(z, 64))
+        ff = max(1, round((count(beside) - base) / step) + 1) * 64
+        models[name] = {"kazepel": dict(measure_design(kazepel_config(z, ff), z["vocab"], args, gen, context, steps), expert_ff=ff),
+                        "katopel": measure_design(beside, z["vocab"], args, gen, context, steps),
+                        "kazepel, layers 2 .. 5 twice": measure_design(kazepel_config(z, ff, (2, 6, 2)), z["vocab"], args, gen,
+                                                                        context, steps)}
+
+    # ---- kernels alone: inputs larger than L2, a 256 MB write between the timed launches ----
+    dev = "cuda:0"
+    flush = torch.empty(64 << 20, dtype=torch.float32, device=dev)
+
+    def kernel_time(fn, reps=7):
+        times = []
+        for _ in range(3 + reps):
+            flush.zero_()
+            ms, _ = timed(fn)
+            times.append(ms)
+        return sorted(times[3:])[reps // 2]
+
+    kernels = {}
+
+    def record(name, ms, nbytes, like, flops=None):
+        kernels[name] = {"us": round(ms * 1e3, 1), "gb_s": round(nbytes / (ms / 1e3) / 1e9), "like": like,
+                         "of_measured_copy_peak": round(nbytes / (ms / 1e3) / 1e9 / pk["hbm_gbs"], 2)}
+        if flops is not None:
+            kernels[name]["tflops"] = round(flops / (ms / 1e3) / 1e12, 1)
+
+    ints = lambda values: torch.tensor(list(values), dtype=torch.int32, device=dev)
+    rnd = lambda *shape, dtype=torch.float32: torch.randn(*shape, device=dev, dtype=torch.float32).to(dtype)
+    T, H, rows = 8192, 2048, 64
+    # ---- both delta rules at the 2k sizes: 16 heads of 128 x 128, 4 taps ----
+    heads, dim, vdim, taps, rank = 16, 128, 128, 4, 128
+    channels = 2 * heads * dim + heads * vdim
+    off = heads * vdim * ops.cdr_padded_dim(dim)
+    slot = off + (taps - 1) * channels
+    proj = rnd(T, channels + 2 * rank + heads + (-(channels + 2 * rank + heads)) % 8)
+    pre = rnd(T, heads * (dim + vdim))
+    conv, a_log, dt_bias = rnd(channels, taps), rnd(heads), rnd(heads * dim)
+    gain_v = torch.ones(vdim, device=dev)
+    o = torch.empty(T, heads * vdim, device=dev)
+    y16 = torch.empty(T, heads * vdim, dtype=torch.bfloat16, device=dev)
+    record_bytes = ops.cdr_record(dim, vdim) * 4
+    d_groups = 8                                          # the Katopel path: 16 heads over 8
+    d_channels = 2 * d_groups * dim + heads * vdim
+    d_off = heads * vdim * ops.gdn_padded_dim(dim)
+    d_slot = -(-(d_off + (taps - 1) * d_channels) // 4) * 4
+    d_proj, d_conv = rnd(T, d_channels + 2 * heads + heads * vdim), rnd(d_channels, taps)
+    qkv, bg = torch.empty(T, d_channels, device=dev), torch.empty(T, 2 * heads + d_groups, device=dev)
+    for requests in (1, 4):
+        spans, slots = ints(T * r // requests for r in range(requests + 1)), ints(range(requests))
+        row_req = ints(r for r in range(requests) for _ in range(T // requests))
+        state = torch.zeros(requests, slot, device=dev)
+        records = ops.cdr_records(T, requests, heads, dim, vdim, dev)
+        where = f"{T} tokens of {requests} request(s)"
+        record(f"cdr_prepare, {where}, {channels} channels of {taps} taps",
+               kernel_time(lambda: ops.cdr_prepare(proj, 0, channels + 2 * rank, pre, heads, heads, dim, vdim, taps, conv, a_log,
+                                                   dt_bias, state, off, spans, slots, records)),
+               T * (channels + heads + heads * dim) * 4 + T // 4 * heads * record_bytes, "gdn_prepare")
+        record(f"cdr_scan, {where}, {heads} heads of {dim} x {vdim}",
+               kernel_time(lambda: ops.cdr_scan(records, heads, dim, vdim, state, spans, slots, o)),
+               T // 4 * heads * record_bytes + T * heads * vdim * 4, "gdn_scan", flops=T * heads * dim * vdim * 8)
+        d_state = torch.zeros(requests, d_slot, device=dev)
+        record(f"gdn_prepare (Katopel path), {where}, {d_channels} channels of {taps} taps",
+               kernel_time(lambda: ops.gdn_prepare(d_proj, 0, d_channels, d_channels + heads, d_groups, heads, dim, vdim, taps, d_conv,
+                                                   a_log, dt_bias, d_state, d_off, row_req, spans, slots, qkv, bg)),
+               T * (d_channels + 2 * heads) * 8, None)
+        record(f"gdn_scan (Katopel path), {where}, {heads} heads of {dim} x {vdim}",
+               kernel_time(lambda: ops.gdn_scan(qkv, bg, d_groups, heads, dim, vdim, d_state, spans, slots, o, longest=T // requests)),
+               T * (d_channels + 2 * heads + heads * vdim) * 4, None, flops=T * heads * dim * vdim * 8)
+    del records, state, d_state
+    row_req = ints([0] * T)
+    record(f"gdn_out_norm with a sigmoid gate, {T} tokens x {heads} heads of {vdim}",
+           kernel_time(lambda: ops.gdn_out_norm(o, pre, heads * dim, gain_v, 1.0, 1e-6, y16, heads, vdim, row_req, gate_kind="sigmoid")),
+           T * heads * vdim * (4 + 4 + 2), "gdn_out_norm")
+    record(f"gdn_out_norm (Katopel path), {T} tokens x {heads} heads of {vdim}",
+           kernel_time(lambda: ops.gdn_out_norm(o, d_proj, d_channels + 2 * heads, gain_v, 1.0, 1e-6, y16, heads, vdim, row_req)),
+           T * heads * vdim * (4 + 4 + 2), None)
+    low = torch.empty(T, 2 * rank, dtype=torch.bfloat16, device=dev)
+    record(f"take_columns, {T} x {2 * rank}", kernel_time(lambda: ops.take_columns(proj, channels, low)), T * 2 * rank * 6, "silu_gate")
+    w2 = rnd(heads * (dim + vdim), 2 * rank, dtype=torch.bfloat16)
+    second = Linear(w2)
+    record(f"the second low-rank products, {T} x {2 * rank} -> {heads * (dim + vdim)} (vendor product, float32 out)",
+           kernel_time(lambda: second.forward(low, out_dtype=torch.float32)), T * heads * (dim + vdim) * 4 + T * 2 * rank * 2, None,
+           flops=T * heads * (dim + vdim) * 4 * rank)
+    spans, slots, req1 = ints(range(rows + 1)), ints(range(rows)), ints(range(rows))
+    state = torch.zeros(rows, slot, device=dev)
+    for inside in (True, False):
+        record(f"cdr_step, {rows} requests of one token, {heads} heads of {dim} x {vdim}, the low-rank products " +
+               ("inside" if inside else "handed in"),
+               kernel_time(lambda: ops.cdr_step(proj[:rows], 0, channels + 2 * rank, channels, rank, rank, w2, None if inside else pre[:rows],
+                                                heads, heads, dim, vdim, taps, conv, a_log, dt_bias, gain_v, 1e-6, state, off, req1,
+                                                slots, True, y16[:rows])), rows * off * 8, "gdn_step")
+    d_state = torch.zeros(rows, d_slot, device=dev)
+    record(f"gdn_step (Katopel path), {rows} requests of one token",
+           kernel_time(lambda: ops.gdn_step(d_proj[:rows], 0, d_channels, d_channels + heads, d_channels + 2 * heads, d_groups, heads,
+                                            dim, vdim, taps, d_conv, a_log, dt_bias, gain_v, 1.0, 1e-6, d_state, d_off, req1, spans, slots,
+                                            y16[:rows])), rows * d_off * 8, None)
+    del state, d_state, proj, pre, d_proj, qkv
+    # ---- the norm, the stream's update, what a pass starts from ----
+    x, y, h16 = rnd(T, H), rnd(T, H, dtype=torch.bfloat16), torch.empty(T, H, dtype=torch.bfloat16, device=dev)
+    g1, b1 = torch.ones(H, device=dev), torch.zeros(H, device=dev)
+    shares = torch.rand(T, 9, device=dev)
+    carried = rnd(T, H, dtype=torch.bfloat16)
+    joined = torch.empty(T, 2 * H, dtype=torch.bfloat16, device=dev)
+    x0 = rnd(T, H)
+    record(f"stream_update with a pending output and the norm, {T} x {H}",
+           kernel_time(lambda: ops.stream_update(x, y, alpha=0.7, gain=g1, bias=b1, out=h16)), T * H * (2 + 4 + 4 + 2), "post_norm_add, rms_norm")
+    record(f"stream_update with a pending output, the input handed through and the norm, {T} x {H}",
+           kernel_time(lambda: ops.stream_update(x, y, carried=carried, share=shares[:, 8], alpha=0.7, gain=g1, bias=b1, out=h16)),
+           T * H * (2 + 2 + 4 + 4 + 2), "post_norm_add, rms_norm")
+    record(f"stream_update into a pass's operand, {T} x {H}",
+           kernel_time(lambda: ops.stream_update(x, y, beside=x0, out=joined)), T * H * (2 + 4 + 4 + 4 + 4), "post_norm_add, rms_norm")
+    record(f"post_norm_add with the next norm (Katopel path), {T} x {H}",
+           kernel_time(lambda: ops.post_norm_add(x, [(y, 1.0)], g1, b1, 1e-6, g1, b1, 1e-6, h16)), T * H * (2 + 4 + 4 + 2), None)
+    record(f"rms_norm with pending add (Qwen2 path), {T} x {H}", kernel_time(lambda: ops.rms_norm(x, g1, 1e-6, h16, delta=y)),
+           T * H * (4 + 4 + 2 + 2), None)
+    del joined, x0, carried
+    # ---- experts ----
+    experts, identity, ff = 8, 4, 704
+    I = experts * ff
+    router = rnd(experts + identity, H)
+    correction = rnd(experts + identity) * 0.01
+    share = torch.empty(T, experts + 1, device=dev)
+    h_in = rnd(T, H, dtype=torch.bfloat16)
+    record(f"moe_route, softmax of all, {experts} experts and {identity} identity ones in 4 groups of which 2, width {H}",
+           kernel_time(lambda: ops.moe_route(h_in, router, experts, 2, None, share, score="softmax", correction=correction, groups=4, keep=2,
+                                             identity=identity, group_worth=1, renormalize=True)), T * H * 2, "moe_route")
+    record(f"moe_route, softmax of the chosen (Katopel path), {experts} experts and a shared one, width {H}",
+           kernel_time(lambda: ops.moe_route(h_in, router[:experts + 1].contiguous(), experts, 2, True, share)), T * H * 2, None)
+    gu, act = rnd(T, 2 * I, dtype=torch.bfloat16), torch.empty(T, I, dtype=torch.bfloat16, device=dev)
+    record(f"moe_gate, clamped, {T} x {I}",
+           kernel_time(lambda: ops.moe_gate(gu, share, act, experts, ff, False, "clamped_swish", limit=7.0, alpha=1.702)), T * I * 6, "moe_gate")
+    record(f"moe_gate, silu (Katopel path), {T} x {I}", kernel_time(lambda: ops.moe_gate(gu, share, act, experts, ff, False)), T * I * 6, None)
+    del gu, act
+    # ---- attention: rotation and cache write; windows with and without kept first tokens ----
+    nh, nkv, d, page = 16, 4, 128, PAGE
+    wide = rnd(T, (nh + 2 * nkv) * d)
+    freq = torch.tensor([1e6 ** (-2.0 * i / 64) for i in range(32)], dtype=torch.float64, device=dev)
+    pos, req = torch.arange(T, dtype=torch.int32, device=dev), torch.zeros(T, dtype=torch.int32, device=dev)
+    bias = torch.zeros((nh + 2 * nkv) * d, device=dev)
+    q_out = torch.empty(T, nh * d, dtype=torch.bfloat16, device=dev)
+    k_pool = torch.zeros(T + 64, nkv, d, dtype=torch.bfloat16, device=dev)
+    v_pool = torch.zeros_like(k_pool)
+    record(f"qkv_rotate_store, the half layout with a factor on cosine and sine, {T} tokens, {nh} heads over {nkv} of {d} lanes, 64 rotated",
+           kernel_time(lambda: ops.qkv_rotate_store(wide, 0, None, freq, 64, pos, pos, req, q_out, k_pool, v_pool, nh, nkv, d, d, d,
+                                                    layout="half", magnitude=1.2)), T * (nh + 2 * nkv) * d * (4 + 2), "qkv_rotate_store")
+    record(f"qkv_rotate_store, biases and the interleaved layout (Katopel path), {T} tokens",
+           kernel_time(lambda: ops.qkv_rotate_store(wide, 0, bias, freq, 64, pos, pos, req, q_out, k_pool, v_pool, nh, nkv, d, d, d)),
+           T * (nh + 2 * nkv) * d * (4 + 2), None)
+    n_req, portion, n_keys, window, keep = 4, 2048, 8192, 1023, 16
+    sink = torch.zeros(nh, device=dev)
+    pages_each = n_keys // page
+    q = rnd(n_req * portion, nh * d, dtype=torch.bfloat16)
+    out = torch.empty_like(q)
+    k_pool, v_pool = rnd(n_req * n_keys, nkv, d, dtype=torch.bfloat16), rnd(n_req * n_keys, nkv, d, dtype=torch.bfloat16)
+    table = torch.arange(n_req * pages_each, dtype=torch.int32, device=dev).view(n_req, pages_each)
+    row_req = torch.arange(n_req, dtype=torch.int32, device=dev).repeat_interleave(portion)
+    pos = (torch.arange(portion, dtype=torch.int32, device=dev) + (n_keys - portion)).repeat(n_req)
+    for kernel, run, tile_rows in (("attention_tcgen05", ops.attention_tcgen05, ops.WIDE_TILE_ROWS),
+                                   ("prefill_attention", ops.prefill_attention, ops.PREFILL_TILE_ROWS)):
+        note = RowTiles(tile_rows)
+        words = np.zeros(note.capacity(n_req * portion, n_req), dtype=np.int32)
+        n_tiles = note.fill(words, np.arange(n_req, dtype=np.int32) * portion, np.full(n_req, portion, dtype=np.int32),
+                            np.full(n_req, n_keys - portion, dtype=np.int32), False)
+        tiles = torch.tensor(words, device=dev).view(-1, 2)
+        for kept in (keep, 0):
+            record(f"{kernel}, {n_req} portions of {portion} rows, a window of 1,024 keys, " +
+                   (f"{keep} first tokens kept and a sink" if kept else "none kept, no sink"),
+                   kernel_time(lambda: run(q, k_pool, v_pool, out, table, row_req, pos, tiles, n_tiles, nh, nkv, d, page, window,
+                                           d ** -0.5, sink=sink if kept else None, keep_first=kept)),
+                   0, kernel + ", none kept" if kept else None, flops=n_req * portion * nh * (1024 + kept) * 4 * d)
+    n_keys = 4096
+    pages_each = n_keys // page
+    big_k, big_v = rnd(rows * n_keys, nkv, d, dtype=torch.bfloat16), rnd(rows * n_keys, nkv, d, dtype=torch.bfloat16)
+    table = torch.arange(rows * pages_each, dtype=torch.int32, device=dev).view(rows, pages_each)
+    q1, req1 = rnd(rows, nh * d, dtype=torch.bfloat16), torch.arange(rows, dtype=torch.int32, device=dev)
+    out1, pos1 = torch.empty_like(q1), torch.full((rows,), n_keys - 1, dtype=torch.int32, device=dev)
+    for kept in (keep, 0):
+        record(f"decode_attention, {rows} rows, a window of 2,048 keys, " + (f"{keep} first tokens kept and a sink" if kept else "none kept, no sink"),
+               kernel_time(lambda: ops.decode_attention(q1, big_k, big_v, out1, table, req1, pos1, nh, nkv, d, page, 2047, d ** -0.5,
+                                                        sink=sink if kept else None, keep_first=kept)),
+               rows * (2048 + kept) * nkv * d * 4, "decode_attention, none kept" if kept else None)
+    ops.raise_if_error()
+    print(json.dumps({
+        "metric": "prefill and decode tok/s of the Kazepel design beside Katopel at equal width, depth and parameters",
+        "unit": "tokens/s", "n_gpus": 1, "steps": steps, "warmup": args.warmup, "dtype": "bf16",
+        "data": "synthetic: random weights drawn on the device, uniform random token ids",
+        "config": {"sizes": KAZEPEL_SIZES, "prefill_tokens": PREFILL_TOKENS, "decode_context": context,
                    "peaks": pk["source"], "hbm_gbs": pk["hbm_gbs"],
                    "l2": "kernels alone: inputs larger than L2 and a 256 MB write between timed launches"},
         "models": models, "kernels": kernels}))
