@@ -425,13 +425,16 @@ cdr_scan_kernel(const float* __restrict__ records, int heads, int vdim, int vdim
 // every head has q and k channels of its own, so the block moves its channels' kept inputs on itself.
 template <typename TW> struct CdrPiece;               // a lane's piece of a weight row: four elements
 template <> struct CdrPiece<float> {
-  static __device__ __forceinline__ float4 load(const float* p) { return *reinterpret_cast<const float4*>(p); }
+  typedef float4 Raw;
+  static __device__ __forceinline__ Raw raw(const float* p) { return *reinterpret_cast<const float4*>(p); }
+  static __device__ __forceinline__ float4 wide(Raw v) { return v; }
 };
 template <> struct CdrPiece<__nv_bfloat16> {
-  static __device__ __forceinline__ float4 load(const __nv_bfloat16* p) {
-    const uint2 raw = *reinterpret_cast<const uint2*>(p);
-    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+  typedef uint2 Raw;
+  static __device__ __forceinline__ Raw raw(const __nv_bfloat16* p) { return *reinterpret_cast<const uint2*>(p); }
+  static __device__ __forceinline__ float4 wide(Raw v) {
+    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
+    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
     return make_float4(lo.x, lo.y, hi.x, hi.y);
   }
 };
@@ -448,7 +451,7 @@ cdr_step_kernel(const float* __restrict__ proj, int ld, int qkv_at, int b_at, in
                 float* __restrict__ state, long long state_stride, int conv_off, const int* __restrict__ row_req,
                 const int* __restrict__ state_slot, int shift, TO* __restrict__ out) {
   constexpr int dim_p = P * DPL, CPT = P / 8;
-  // q, k, g [dim_p] each; v, o, gate [vdim] each; low-rank activations [ra + rg]
+  // q, k [dim_p] each, v [vdim], decays [dim_p], o, gate [vdim] each; low-rank activations [ra + rg]
   extern __shared__ __align__(16) float cdr_one[];
   __shared__ float scratch[33], misc[4];
   const int t = blockIdx.x, h = blockIdx.y;
@@ -457,9 +460,9 @@ cdr_step_kernel(const float* __restrict__ proj, int ld, int qkv_at, int b_at, in
   const int part = lane % P, group = lane / P;
   float* q_s = cdr_one;
   float* k_s = q_s + dim_p;
-  float* g_s = k_s + dim_p;
-  float* v_s = g_s + dim_p;
-  float* o_s = v_s + vdim;
+  float* v_s = k_s + dim_p;
+  float* g_s = v_s + vdim;
+  float* o_s = g_s + dim_p;
   float* gate_s = o_s + vdim;
   float* low_s = gate_s + (vdim + (-(3 * vdim) & 3));         // on 16 bytes
   float* slot = state + (size_t)(r < 0 ? 0 : state_slot[r]) * state_stride;
@@ -478,61 +481,110 @@ cdr_step_kernel(const float* __restrict__ proj, int ld, int qkv_at, int b_at, in
     }
   };
   const int my_col = warp * 4 + group * CPT;
-  if (r >= 0) load_columns(my_col);
+  const int g = h / (heads / groups);
+  const int channels = 2 * groups * dim + heads * vdim;
+  float* kept = slot + conv_off;
+  // ... and so are the thread's first channel's taps and kept inputs, and the warp's first rows of the second
+  // products (a lane's first four elements of each), which nothing of this step writes
+  constexpr int kAhead = 8;
+  const int outputs = dim_p + vdim;
+  auto second_row = [&](int i) {               // the weight row of output i and where its inputs start; null: none
+    const bool decay = i < dim_p;
+    const int l = decay ? i : i - dim_p;
+    return decay && l >= dim ? (const TW*)nullptr
+                             : w2 + (size_t)(decay ? h * dim + l : heads * dim + h * vdim + l) * (ra + rg) + (decay ? 0 : ra);
+  };
+  auto channel_of = [&](int i) {               // the channel of item i of q, k, v; -1: a padded lane
+    if (i >= 2 * dim_p) return 2 * groups * dim + h * vdim + i - 2 * dim_p;
+    const int l = i < dim_p ? i : i - dim_p;
+    return l < dim ? (i < dim_p ? g : groups + g) * dim + l : -1;
+  };
+  float tap[4], old[3];
+  typename CdrPiece<TW>::Raw ahead[kAhead];
+  const int first_channel = (int)threadIdx.x < 2 * dim_p + vdim ? channel_of(threadIdx.x) : -1;
+  const bool quick = taps == 4 && first_channel >= 0;
+  if (r >= 0) {
+    load_columns(my_col);
+    if (quick) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) tap[j] = conv_w[(size_t)first_channel * 4 + j];
+#pragma unroll
+      for (int j = 0; j < 3; ++j) old[j] = kept[(size_t)j * channels + first_channel];
+    }
+    if (pre == nullptr) {
+#pragma unroll
+      for (int k = 0; k < kAhead; ++k) {
+        const int i = warp + k * warps;
+        const TW* w = i < outputs ? second_row(i) : nullptr;
+        if (w != nullptr && lane * 4 < (i < dim_p ? ra : rg)) ahead[k] = CdrPiece<TW>::raw(w + lane * 4);
+      }
+    }
+  }
   pdl_wait();
   pdl_launch();
   if (r < 0) return;
-  const int g = h / (heads / groups);
-  const int channels = 2 * groups * dim + heads * vdim;
   const float* row = proj + (size_t)t * ld;
-  float* kept = slot + conv_off;
   for (int i = threadIdx.x; i < 2 * dim_p + vdim; i += blockDim.x) {
-    const int which = i < dim_p ? 0 : i < 2 * dim_p ? 1 : 2;
-    const int l = i - which * dim_p;
+    const int c = channel_of(i);
     float value = 0.f;
-    if (which == 2 || l < dim) {
-      const int c = which == 0 ? g * dim + l : which == 1 ? (groups + g) * dim + l : 2 * groups * dim + h * vdim + l;
+    if (c >= 0) {
       const float newest = row[qkv_at + c];
-      float acc = conv_w[(size_t)c * taps + taps - 1] * newest;
-      for (int j = 0; j + 1 < taps; ++j) {
-        const float in = kept[(size_t)j * channels + c];
-        acc = fmaf(conv_w[(size_t)c * taps + j], in, acc);
-        if (shift && j > 0) kept[(size_t)(j - 1) * channels + c] = in;
+      float acc;
+      if (quick && i == (int)threadIdx.x) {
+        acc = tap[3] * newest;
+#pragma unroll
+        for (int j = 0; j < 3; ++j) acc = fmaf(tap[j], old[j], acc);
+        if (shift) {
+          kept[c] = old[1];
+          kept[(size_t)channels + c] = old[2];
+        }
+      } else {
+        acc = conv_w[(size_t)c * taps + taps - 1] * newest;
+        for (int j = 0; j + 1 < taps; ++j) {                // kept inputs move on one place as they are read
+          const float in = kept[(size_t)j * channels + c];
+          acc = fmaf(conv_w[(size_t)c * taps + j], in, acc);
+          if (shift && j > 0) kept[(size_t)(j - 1) * channels + c] = in;
+        }
       }
       if (shift && taps > 1) kept[(size_t)(taps - 2) * channels + c] = newest;
       value = acc * cdr_sigmoid(acc);
     }
-    (which == 0 ? q_s : which == 1 ? k_s : v_s)[l] = value;
+    q_s[i] = value;                            // q, k and v lie one behind the other
   }
   if (pre == nullptr)
     for (int i = threadIdx.x; i < ra + rg; i += blockDim.x) low_s[i] = row[low_at + i];
   __syncthreads();
   // the decay's and the gate's second products (a warp an output), and the token's unit vectors
   const float a = expf(a_log[h]);
-  const int outputs = dim_p + vdim;
   if (pre == nullptr) {
-    for (int i = warp; i < outputs; i += warps) {
-      const bool decay = i < dim_p;
-      const int l = decay ? i : i - dim_p;
-      if (decay && l >= dim) {
-        if (lane == 0) g_s[l] = 1.f;
-        continue;
+    // kAhead outputs a warp at a time, so that their sums cross the lanes side by side; lane k finishes output k
+    for (int base = warp; base < outputs; base += kAhead * warps) {
+      float acc[kAhead];
+#pragma unroll
+      for (int k = 0; k < kAhead; ++k) {
+        const int i = base + k * warps;
+        const TW* w = i < outputs ? second_row(i) : nullptr;
+        const int from = i < dim_p ? 0 : ra, n = w == nullptr ? 0 : i < dim_p ? ra : rg;
+        acc[k] = 0.f;
+        for (int j = lane * 4; j < n; j += 128) {        // ranks and their sum are whole 8s
+          const float4 x = CdrPiece<TW>::wide(base == warp && j < 128 ? ahead[k] : CdrPiece<TW>::raw(w + j));
+          const float4 y = *reinterpret_cast<const float4*>(low_s + from + j);
+          acc[k] = fmaf(x.x, y.x, acc[k]);
+          acc[k] = fmaf(x.y, y.y, acc[k]);
+          acc[k] = fmaf(x.z, y.z, acc[k]);
+          acc[k] = fmaf(x.w, y.w, acc[k]);
+        }
       }
-      const int from = decay ? 0 : ra, n = decay ? ra : rg;
-      const TW* w = w2 + (size_t)(decay ? h * dim + l : heads * dim + h * vdim + l) * (ra + rg) + from;
-      float acc = 0.f;
-      for (int j = lane * 4; j < n; j += 128) {          // ranks and their sum are whole 8s
-        const float4 x = CdrPiece<TW>::load(w + j);
-        const float4 y = *reinterpret_cast<const float4*>(low_s + from + j);
-        acc = fmaf(x.x, y.x, acc);
-        acc = fmaf(x.y, y.y, acc);
-        acc = fmaf(x.z, y.z, acc);
-        acc = fmaf(x.w, y.w, acc);
+      float mine = 0.f;
+#pragma unroll
+      for (int k = 0; k < kAhead; ++k) {
+        acc[k] = warp_sum(acc[k]);
+        if (lane == k) mine = acc[k];
       }
-      acc = warp_sum(acc);
-      if (lane == 0) {
-        if (decay) g_s[l] = expf(-a * cdr_softplus(acc + dt_bias[h * dim + l]));
-        else gate_s[l] = cdr_sigmoid(acc);
+      const int i = base + lane * warps;
+      if (lane < kAhead && i < outputs) {
+        if (i >= dim_p) gate_s[i - dim_p] = cdr_sigmoid(mine);
+        else g_s[i] = i < dim ? expf(-a * cdr_softplus(mine + dt_bias[h * dim + i])) : 1.f;
       }
     }
   } else {

@@ -101,103 +101,133 @@ __device__ __forceinline__ void moe_choose(const float* z, const float* choice, 
   }
 }
 
+// One warp: the softmax over the `top` largest logits alone, zero elsewhere (ties: the lower index).
+__device__ __forceinline__ void moe_softmax_of_chosen(const float* z, float* out, int experts, int top, int columns, int lane) {
+  unsigned taken = 0u;                                  // bit i: expert lane + 32 i
+  float highest = 0.f, sum = 0.f;
+  for (int c = lane; c < columns; c += 32) out[c] = 0.f;
+  for (int k = 0; k < top; ++k) {
+    int best = -1;
+    float value = -INFINITY;
+    for (int e = lane, i = 0; e < experts; e += 32, ++i)
+      if (!((taken >> i) & 1u) && (best < 0 ? z[e] == z[e] : z[e] > value)) {
+        best = e;
+        value = z[e];
+      }
+    moe_warp_best(value, best);
+    if (best < 0) break;
+    if (k == 0) highest = value;
+    sum += expf(value - highest);
+    if (best % 32 == lane) taken |= 1u << (best / 32);
+  }
+  __syncwarp();
+  for (int e = lane, i = 0; e < experts; e += 32, ++i)
+    if ((taken >> i) & 1u) out[e] = expf(z[e] - highest) / sum;
+}
+
+__device__ __forceinline__ float4 moe_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 moe_load4(const __nv_bfloat16* p) {
+  const uint2 raw = *reinterpret_cast<const uint2*>(p);
+  const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+  const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+  return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+
+#define MOE_TOKENS 8       // tokens a block takes where there are many: every router row is then read once for eight
+
 // `experts` counts every router output that is chosen among, the `identity` last ones included.
 // h: the feed-forward's input [T, hidden] (float32, or its bfloat16 rounding); w: float32
 // [experts + shared, hidden], the router's rows and behind them the shared expert's gate row.
-// A block a token: its warps take the logits in turn (32-bit sums), thread 0 then chooses.
-template <typename TI>
-__global__ void __launch_bounds__(128)
-moe_route_kernel(const TI* __restrict__ h, const float* __restrict__ w, int hidden, int experts, int top,
+// A block takes TOK tokens: its warps take the logits in turn (32-bit sums, a lane's share of a token's sum
+// and the order in which the shares meet do not depend on TOK), then a warp a token chooses.
+template <typename TI, int TOK>
+__global__ void __launch_bounds__(TOK == 1 ? 1024 : 256, 1)
+moe_route_kernel(const TI* __restrict__ h, const float* __restrict__ w, int n_rows, int hidden, int experts, int top,
                  int shared_mode, float* __restrict__ share, int score, const float* __restrict__ correction,
                  int groups, int keep, float scale, int identity, int worth, int renormalize) {
-  __shared__ float z[MOE_MAX_EXPERTS + 1];
-  __shared__ float choice[MOE_MAX_EXPERTS], group_worth[MOE_MAX_EXPERTS];
-  __shared__ float scratch[33];
-  __shared__ unsigned char open[MOE_MAX_EXPERTS];                  // groups whose experts may be chosen
+  // a token: logits (then scores) and the shared expert's, choice scores, the groups' worth, the open groups
+  extern __shared__ float moe_s[];
   const int shared = shared_mode == MOE_SHARED_GATED ? 1 : 0;      // router rows behind the experts'
-  const int real = experts - identity;
+  const int real = experts - identity, outputs = experts + shared;
   const int columns = real + (shared_mode != MOE_SHARED_NONE ? 1 : 0) + (identity > 0 ? 1 : 0);
+  const int per_token = 2 * experts + 1 + 2 * groups;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  const int t0 = blockIdx.x * TOK;
+  if (TOK == 1) {            // few tokens: the router's rows towards L2 while the predecessor runs
+    const size_t bytes = (size_t)outputs * hidden * sizeof(float);
+    for (size_t at = (size_t)threadIdx.x * 128; at < bytes; at += (size_t)blockDim.x * 128)
+      asm volatile("prefetch.global.L2 [%0];" ::"l"(reinterpret_cast<const char*>(w) + at));
+  }
   pdl_wait();
   pdl_launch();
-  const int t = blockIdx.x;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const TI* row = h + (size_t)t * hidden;
-  for (int e = warp; e < experts + shared; e += blockDim.x >> 5) {
+  const bool wide = hidden % 128 == 0 && ((((uintptr_t)h) | ((uintptr_t)w)) & 15) == 0;
+  const TI* rows[TOK];
+#pragma unroll
+  for (int i = 0; i < TOK; ++i) rows[i] = h + (size_t)(t0 + i < n_rows ? t0 + i : t0) * hidden;
+  for (int e = warp; e < outputs; e += warps) {
     const float* we = w + (size_t)e * hidden;
-    float acc = 0.f;
-    if (hidden % 128 == 0 && ((((uintptr_t)row) | ((uintptr_t)we)) & 15) == 0) {
-      // four consecutive elements a lane and trip: one load of the input's, one of the router's row
-      for (int i = lane * 4; i < hidden; i += 128) {
-        const float4 wv = *reinterpret_cast<const float4*>(we + i);
-        float4 hv;
-        if (sizeof(TI) == 4) {
-          hv = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(row) + i);
-        } else {
-          const uint2 raw = *reinterpret_cast<const uint2*>(reinterpret_cast<const __nv_bfloat16*>(row) + i);
-          const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-          const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-          hv = make_float4(lo.x, lo.y, hi.x, hi.y);
+    float acc[TOK];
+#pragma unroll
+    for (int i = 0; i < TOK; ++i) acc[i] = 0.f;
+    if (wide) {
+      // four consecutive elements a lane and trip
+#pragma unroll (TOK == 1 ? 8 : 2)
+      for (int c = lane * 4; c < hidden; c += 128) {
+        const float4 wv = moe_load4(we + c);
+#pragma unroll
+        for (int i = 0; i < TOK; ++i) {
+          const float4 hv = moe_load4(rows[i] + c);
+          acc[i] = fmaf(hv.x, wv.x, acc[i]);
+          acc[i] = fmaf(hv.y, wv.y, acc[i]);
+          acc[i] = fmaf(hv.z, wv.z, acc[i]);
+          acc[i] = fmaf(hv.w, wv.w, acc[i]);
         }
-        acc = fmaf(hv.x, wv.x, acc);
-        acc = fmaf(hv.y, wv.y, acc);
-        acc = fmaf(hv.z, wv.z, acc);
-        acc = fmaf(hv.w, wv.w, acc);
       }
-    } else
-    for (int i = lane; i < hidden; i += 32) acc = fmaf(to_float(row[i]), we[i], acc);
-    acc = warp_sum(acc);
-    if (lane == 0) z[e] = acc;
+    } else {
+      for (int c = lane; c < hidden; c += 32) {
+        const float wv = we[c];
+#pragma unroll
+        for (int i = 0; i < TOK; ++i) acc[i] = fmaf(to_float(rows[i][c]), wv, acc[i]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < TOK; ++i) {
+      const float sum = warp_sum(acc[i]);
+      if (lane == 0) moe_s[i * per_token + e] = sum;
+    }
   }
   __syncthreads();
+  const int t = t0 + warp;
+  if (warp >= TOK || t >= n_rows) return;
+  float* z = moe_s + warp * per_token;
+  float* choice = z + experts + 1;
+  float* group_worth = choice + experts;
+  unsigned char* open = reinterpret_cast<unsigned char*>(group_worth + groups);
   float* out = share + (size_t)t * columns;
-  if (score != MOE_SCORE_SOFTMAX_OF_CHOSEN) {
+  if (score == MOE_SCORE_SOFTMAX_OF_CHOSEN) {
+    moe_softmax_of_chosen(z, out, experts, top, columns, lane);
+  } else {
     float highest = 0.f, total = 1.f;
     if (score == MOE_SCORE_SOFTMAX) {
-      float m = -INFINITY, sum = 0.f;
-      for (int e = threadIdx.x; e < experts; e += blockDim.x) m = fmaxf(m, z[e]);
-      highest = block_max(m, scratch);
-      for (int e = threadIdx.x; e < experts; e += blockDim.x) sum += expf(z[e] - highest);
-      total = block_sum(sum, scratch);
+      highest = -INFINITY;
+      for (int e = lane; e < experts; e += 32) highest = fmaxf(highest, z[e]);
+      highest = warp_max(highest);
+      total = 0.f;
+      for (int e = lane; e < experts; e += 32) total += expf(z[e] - highest);
+      total = warp_sum(total);
     }
-    for (int e = threadIdx.x; e < experts; e += blockDim.x) {
+    for (int e = lane; e < experts; e += 32) {
       const float s = score == MOE_SCORE_SOFTMAX ? expf(z[e] - highest) / total : 1.0f / (1.0f + expf(-z[e]));
       z[e] = s;
       choice[e] = s + (correction ? correction[e] : 0.f);
     }
-    __syncthreads();
-    if (warp != 0) return;
+    __syncwarp();
     moe_choose(z, choice, group_worth, open, out, experts, real, identity, top, groups, keep, worth, renormalize, scale,
                columns, lane);
-    if (lane == 0 && shared_mode == MOE_SHARED_ONE) out[real] = 1.0f;
-    if (lane == 0 && shared_mode == MOE_SHARED_GATED) out[real] = 1.0f / (1.0f + expf(-z[experts]));
-    return;
   }
-  for (int e = threadIdx.x; e < experts; e += blockDim.x) out[e] = 0.f;
-  __syncthreads();
-  if (threadIdx.x != 0) return;
-  unsigned taken[MOE_MAX_EXPERTS / 32];
-  for (int i = 0; i < (experts + 31) / 32; ++i) taken[i] = 0u;
-  float highest = 0.f, sum = 0.f;
-  for (int k = 0; k < top; ++k) {
-    int best = -1;
-    float value = -INFINITY;
-    for (int e = 0; e < experts; ++e) {
-      if (!((taken[e >> 5] >> (e & 31)) & 1u) && (best < 0 ? z[e] == z[e] : z[e] > value)) {
-        best = e;
-        value = z[e];
-      }
-    }
-    if (best < 0) break;
-    taken[best >> 5] |= 1u << (best & 31);
-    if (k == 0) highest = value;
-    const float weight = expf(value - highest);
-    out[best] = weight;
-    sum += weight;
-  }
-  for (int e = 0; e < experts; ++e)
-    if ((taken[e >> 5] >> (e & 31)) & 1u) out[e] /= sum;
-  if (shared_mode == MOE_SHARED_GATED) out[experts] = 1.0f / (1.0f + expf(-z[experts]));
-  if (shared_mode == MOE_SHARED_ONE) out[experts] = 1.0f;
+  __syncwarp();
+  if (lane == 0 && shared_mode == MOE_SHARED_ONE) out[real] = 1.0f;
+  if (lane == 0 && shared_mode == MOE_SHARED_GATED) out[real] = 1.0f / (1.0f + expf(-z[experts]));
 }
 
 // act(gate) * up of one inner lane: the activations of every gated feed-forward, and the clamped one
@@ -283,13 +313,26 @@ TOKB200_API int tokb200_moe_route(const void* h, int h_dtype, const float* w, in
       score < MOE_SCORE_SOFTMAX_OF_CHOSEN || score > MOE_SCORE_SOFTMAX || groups <= 0 || experts % groups ||
       keep <= 0 || keep > groups || (long long)keep * (experts / groups) < top)
     return TOKB200_BAD_SIZE;
-  if (h_dtype == TOKB200_F32)
-    return launch_dependent(moe_route_kernel<float>, dim3(n_rows), dim3(128), 0, stream, (const float*)h, w, hidden,
-                            experts, top, shared, share, score, correction, groups, keep, scale, identity, worth, renormalize);
-  if (h_dtype == TOKB200_BF16)
-    return launch_dependent(moe_route_kernel<__nv_bfloat16>, dim3(n_rows), dim3(128), 0, stream,
-                            (const __nv_bfloat16*)h, w, hidden, experts, top, shared, share, score, correction, groups,
-                            keep, scale, identity, worth, renormalize);
+  const int outputs = experts + (shared == MOE_SHARED_GATED ? 1 : 0);
+  const size_t per_token = (size_t)(2 * experts + 1 + 2 * groups) * sizeof(float);
+  // many tokens of a router that is not large: eight a block; else one a block, a warp an output
+  const bool many = n_rows > 148 && MOE_TOKENS * per_token <= 48 * 1024;
+  const int warps = outputs < 4 ? 4 : outputs < 32 ? outputs : 32;
+  const dim3 grid(many ? (n_rows + MOE_TOKENS - 1) / MOE_TOKENS : n_rows), block(many ? 256 : warps * 32);
+  const size_t smem = per_token * (many ? MOE_TOKENS : 1);
+#define LAUNCH(TI, TOK)                                                                                           \
+  return launch_dependent(moe_route_kernel<TI, TOK>, grid, block, smem, stream, (const TI*)h, w, n_rows, hidden,   \
+                          experts, top, shared, share, score, correction, groups, keep, scale, identity, worth,    \
+                          renormalize)
+  if (h_dtype == TOKB200_F32) {
+    if (many) LAUNCH(float, MOE_TOKENS);
+    LAUNCH(float, 1);
+  }
+  if (h_dtype == TOKB200_BF16) {
+    if (many) LAUNCH(__nv_bfloat16, MOE_TOKENS);
+    LAUNCH(__nv_bfloat16, 1);
+  }
+#undef LAUNCH
   return TOKB200_BAD_DTYPE;
 }
 

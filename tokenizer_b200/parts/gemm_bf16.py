@@ -64,8 +64,9 @@ def use_pair(M: int, N: int, K: int) -> bool:
     """Many rows, a long k and enough tiles of 256 x 256 for most of a device's 74 pairs of SMs
     (the down projection from 2,816 rows on, where tiles of 128 x 128 need a second round of
     CTAs and take 48 us at 3,072 rows): the product goes to pairs of CTAs, each loading half of
-    the weight tile."""
-    return ops._PAIR and K >= 2048 and N % 8 == 0 and -(-M // 256) * -(-N // 256) >= (sm_count() // 2) * 3 // 5
+    the weight tile.  A weight of many rows has that many tiles with a single row of tokens; up to 128
+    rows fill half a tile at most, and the kernels for few rows take them."""
+    return ops._PAIR and M > 128 and K >= 2048 and N % 8 == 0 and -(-M // 256) * -(-N // 256) >= (sm_count() // 2) * 3 // 5
 
 
 def use_pair_halves(M: int, N: int, K: int) -> bool:
