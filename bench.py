@@ -1668,8 +1668,12 @@ def run_kazepel(args):
     record(f"gdn_out_norm (Katopel path), {T} tokens x {heads} heads of {vdim}",
            kernel_time(lambda: ops.gdn_out_norm(o, d_proj, d_channels + 2 * heads, gain_v, 1.0, 1e-6, y16, heads, vdim, row_req)),
            T * heads * vdim * (4 + 4 + 2), None)
-    low = torch.empty(T, 2 * rank, dtype=torch.bfloat16, device=dev)
-    record(f"take_columns, {T} x {2 * rank}", kernel_time(lambda: ops.take_columns(proj, channels, low)), T * 2 * rank * 6, "silu_gate")
+    many = rnd(8 * T, 1024)                              # eight times the rows: the columns of T alone would fit L2
+    low = torch.empty(8 * T, 2 * rank, dtype=torch.bfloat16, device=dev)
+    record(f"take_columns, {2 * rank} columns of {8 * T} rows", kernel_time(lambda: ops.take_columns(many, 512, low)),
+           8 * T * 2 * rank * 6, "gdn_out_norm")
+    del many
+    low = low[:T]
     w2 = rnd(heads * (dim + vdim), 2 * rank, dtype=torch.bfloat16)
     second = Linear(w2)
     record(f"the second low-rank products, {T} x {2 * rank} -> {heads * (dim + vdim)} (vendor product, float32 out)",

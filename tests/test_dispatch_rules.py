@@ -59,4 +59,5 @@ def test_the_sizes_the_rules_were_measured_at():
     assert rules.choose_tile_k_splits(2048, 896, 4864) == 1          # planes of 7.3 MB: not on lone CTAs
     assert rules.use_pair_halves(2048, 896, 4864) and not rules.use_pair(2048, 896, 4864)
     assert rules.use_pair(4096, 896, 4864) and not rules.use_pair_halves(4096, 896, 4864)
+    assert not rules.use_pair(1, 22528, 2048) and not rules.use_pair(128, 22528, 2048) and rules.use_pair(256, 22528, 2048)
     assert not rules.use_pair(2048, 896, 896) and not rules.use_pair_halves(2048, 1152, 896)

@@ -434,6 +434,15 @@ def test_a_step_of_single_tokens_in_one_kernel(groups, heads, dim, vdim, taps, o
     assert float(one[3].abs().max()) > 0 and float(one[2].abs().max()) == 0
 
 
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("rows,width,at,n", [(5, 40, 8, 16), (300, 64, 4, 48), (7, 37, 3, 9), (1, 24, 6, 16)])
+def test_columns_of_a_product_in_the_compute_type(rows, width, at, n, dtype):
+    proj = rnd(rows, width, seed=5)
+    out = torch.full((rows, n), float("nan"), dtype=dtype, device=DEV)
+    ops().take_columns(proj, at, out)
+    assert torch.equal(out, proj[:, at:at + n].to(dtype))
+
+
 @pytest.mark.parametrize("dim", [32, 64, 128, 256])
 def test_a_channel_without_decay_keeps_what_was_written_far_back(dim):
     """Channel 0 never decays, all others lose everything each token: what token 3 wrote along a key of both comes

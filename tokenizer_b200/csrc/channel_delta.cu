@@ -662,6 +662,26 @@ __global__ void take_columns_kernel(const float* __restrict__ proj, int ld, int 
     out[i] = from_float<TO>(proj[(i / n) * ld + at + i % n]);
 }
 
+// columns and rows in whole 8s, everything on 16 bytes: eight consecutive columns a thread
+__device__ __forceinline__ void take_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void take_store4(__nv_bfloat16* p, float4 v) {
+  __nv_bfloat162 h[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
+  *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(h);
+}
+template <typename TO>
+__global__ void take_columns8_kernel(const float* __restrict__ proj, int ld, int at, int n8, TO* __restrict__ out, int n_rows) {
+  pdl_wait();
+  pdl_launch();
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n_rows * n8) return;
+  const int t = i / n8, c = (i - t * n8) * 8;
+  const float* in = proj + (size_t)t * ld + at + c;
+  const float4 a = *reinterpret_cast<const float4*>(in), b = *reinterpret_cast<const float4*>(in + 4);
+  TO* o = out + (size_t)t * n8 * 8 + c;
+  take_store4(o, a);
+  take_store4(o + 4, b);
+}
+
 // ---- launchers -----------------------------------------------------------------------------------------
 static inline int cdr_parts(int dim) { return dim <= 32 ? 8 : dim <= 64 ? 16 : 32; }
 static inline int cdr_rows(int dim) { return dim <= 128 ? 4 : dim <= 256 ? 8 : 16; }
@@ -777,6 +797,15 @@ TOKB200_API int tokb200_take_columns(const float* proj, int ld, int at, int n, v
   if (n_rows <= 0 || n <= 0) return TOKB200_OK;
   if (at < 0 || at + n > ld) return TOKB200_BAD_SIZE;
   const size_t total = (size_t)n_rows * n, blocks = (total + 255) / 256;
+  if (n % 8 == 0 && at % 4 == 0 && ld % 4 == 0 && ((((uintptr_t)proj) | ((uintptr_t)out)) & 15) == 0 &&
+      total / 8 < (1u << 30)) {
+    const dim3 wide((unsigned)((total / 8 + 255) / 256));
+    if (out_dtype == TOKB200_F32)
+      return launch_dependent(take_columns8_kernel<float>, wide, dim3(256), 0, stream, proj, ld, at, n / 8, (float*)out, n_rows);
+    if (out_dtype == TOKB200_BF16)
+      return launch_dependent(take_columns8_kernel<__nv_bfloat16>, wide, dim3(256), 0, stream, proj, ld, at, n / 8,
+                              (__nv_bfloat16*)out, n_rows);
+  }
   const dim3 grid((unsigned)(blocks < 8192 ? blocks : 8192));
   if (out_dtype == TOKB200_F32)
     return launch_dependent(take_columns_kernel<float>, grid, dim3(256), 0, stream, proj, ld, at, n, (float*)out, total);
