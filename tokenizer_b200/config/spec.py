@@ -90,10 +90,14 @@ class ModelSpec:
     order: Tuple[LayerCall, ...]
     final_norm: PartSpec
     head: PartSpec
+    # how many residual streams run side by side (the layers' blocks then connect to all of them); None: one, plain
+    streams: Optional[int] = None
 
     def validate(self) -> None:
         if not self.layers or not self.order:
             raise ConfigError("a model needs at least one layer and one call in its order")
+        if self.streams is not None and (self.streams < 1 or any(call.before is not None for call in self.order)):
+            raise ConfigError("a model has at least one stream; what enters between layers knows one stream only")
         for at, call in enumerate(self.order):
             if not 0 <= call.layer < len(self.layers):
                 raise ConfigError(f"order[{at}] names layer {call.layer}, there are {len(self.layers)}")

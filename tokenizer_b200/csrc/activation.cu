@@ -8,6 +8,8 @@
 // output (possibly float32 partial sums of a product cut along k, possibly still lacking its
 // bias) times the gate whose pre-activation a projection of the sublayer's input produced.
 // The result is float32: it is what the residual stream adds.
+//
+// activate: the activation of a dense feed-forward, element by element.
 #include "common.cuh"
 
 // The three sums of a block in one pass over shared memory.
@@ -390,5 +392,49 @@ TOKB200_API int tokb200_gated_add_rms_norm(float* x, const void* y, int y_dtype,
   if (y_dtype == TOKB200_BF16 && out_dtype == TOKB200_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);
   if (y_dtype == TOKB200_BF16 && out_dtype == TOKB200_F32) LAUNCH(__nv_bfloat16, float);
 #undef LAUNCH
+  return TOKB200_BAD_DTYPE;
+}
+
+// ---- the activation of a dense feed-forward as a kernel of its own -------------------------
+// out = act(z), element by element; out may be z (for products whose own kernel has no epilogue for it).
+template <typename T>
+__global__ void activate_kernel(const T* z, T* out, int act, size_t n) {
+  pdl_wait();
+  pdl_launch();
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x)
+    out[i] = from_float<T>(gate_activation(act, to_float(z[i])));
+}
+
+// bfloat16, eight neighbours a thread
+__global__ void __launch_bounds__(256)
+activate_bf16x8_kernel(const __nv_bfloat16* z, __nv_bfloat16* out, int act, size_t n8) {
+  pdl_wait();
+  pdl_launch();
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n8; i += (size_t)gridDim.x * blockDim.x) {
+    uint4 raw = reinterpret_cast<const uint4*>(z)[i];
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 v = __bfloat1622float2(h[e]);
+      h[e] = __floats2bfloat162_rn(gate_activation(act, v.x), gate_activation(act, v.y));
+    }
+    reinterpret_cast<uint4*>(out)[i] = raw;
+  }
+}
+
+TOKB200_API int tokb200_activate(const void* z, void* out, int dtype, int act, long long n, cudaStream_t stream) {
+  if (n <= 0) return TOKB200_OK;
+  if (act < 0 || act >= TOKB200_ACT_COUNT) return TOKB200_BAD_SIZE;
+  const bool wide = dtype == TOKB200_BF16 && n % 8 == 0 && (((uintptr_t)z | (uintptr_t)out) & 15) == 0;
+  const size_t items = (size_t)(wide ? n / 8 : n), blocks = (items + 255) / 256;
+  const dim3 grid((unsigned)(blocks < 148 * 16 ? blocks : 148 * 16));
+  if (wide)
+    return launch_dependent(activate_bf16x8_kernel, grid, dim3(256), 0, stream, (const __nv_bfloat16*)z,
+                            (__nv_bfloat16*)out, act, items);
+  if (dtype == TOKB200_BF16)
+    return launch_dependent(activate_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)z,
+                            (__nv_bfloat16*)out, act, items);
+  if (dtype == TOKB200_F32)
+    return launch_dependent(activate_kernel<float>, grid, dim3(256), 0, stream, (const float*)z, (float*)out, act, items);
   return TOKB200_BAD_DTYPE;
 }

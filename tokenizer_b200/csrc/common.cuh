@@ -146,11 +146,12 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_float<__nv_bfloat16>(f
   return __float2bfloat16_rn(v);
 }
 
-// ---- the activation of a gated feed-forward -------------------------------------------
-// out = act(gate) * up.  Which activation is a PARAMETER of every kernel that applies one
-// (the separate gate kernels, the epilogues of the gated products, the fused feed-forward),
-// computed in 32-bit; the tags are shared with Python.
-enum : int { TOKB200_ACT_SILU = 0, TOKB200_ACT_GELU_TANH = 1, TOKB200_ACT_RELU = 2, TOKB200_ACT_COUNT = 3 };
+// ---- the activation of a feed-forward ---------------------------------------------------
+// Gated: out = act(gate) * up; dense: out = act(up).  Which activation is a PARAMETER of every kernel that applies one
+// (the separate gate kernels, the epilogues of the gated and of the plain products, the fused feed-forward),
+// computed in 32-bit; the tags are shared with Python.  NONE: a plain product's result as it is.
+enum : int { TOKB200_ACT_NONE = -1, TOKB200_ACT_SILU = 0, TOKB200_ACT_GELU_TANH = 1, TOKB200_ACT_RELU = 2,
+             TOKB200_ACT_RELU_SQUARED = 3, TOKB200_ACT_COUNT = 4 };
 
 __device__ __forceinline__ float gate_activation(int kind, float g) {
   if (kind == TOKB200_ACT_SILU) return g / (1.0f + expf(-g));            // z * sigmoid(z)
@@ -158,7 +159,8 @@ __device__ __forceinline__ float gate_activation(int kind, float g) {
     const float inner = 0.7978845608028654f * (g + 0.044715f * g * g * g);
     return 0.5f * g * (1.0f + tanhf(inner));
   }
-  return fmaxf(g, 0.f);
+  const float up = fmaxf(g, 0.f);
+  return kind == TOKB200_ACT_RELU_SQUARED ? up * up : up;
 }
 
 // The first key a query at position p sees: 0; p - window where the layer has a window (window >= 0:

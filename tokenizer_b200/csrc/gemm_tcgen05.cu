@@ -357,7 +357,7 @@ struct TcPersistentSmem {
 // What the epilogues need besides the product.  QKV: each row's position and cache slot, the
 // rotary tables, the key/value pools and the head geometry.  GATED: the activation's tag.
 struct QkvEpilogue {
-  int activation;               // the gated epilogue's activation (TOKB200_ACT_*)
+  int activation;               // the epilogue's activation (TOKB200_ACT_*): of a gated product, or of a plain bfloat16 one
   const int* pos;
   const int* slot;              // may be null: no cache write
   const float* cos_t;
@@ -647,8 +647,12 @@ gemm_tcgen05_persistent_kernel(const __grid_constant__ CUtensorMap map_x,
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
               const int col = n0 + c0 + 8 * j + 2 * e;
-              const float lo = __uint_as_float(v[8 * j + 2 * e]) + (bias && col < N ? bias[col] : 0.f);
-              const float hi = __uint_as_float(v[8 * j + 2 * e + 1]) + (bias && col + 1 < N ? bias[col + 1] : 0.f);
+              float lo = __uint_as_float(v[8 * j + 2 * e]) + (bias && col < N ? bias[col] : 0.f);
+              float hi = __uint_as_float(v[8 * j + 2 * e + 1]) + (bias && col + 1 < N ? bias[col + 1] : 0.f);
+              if (!QKV && qkv.activation != TOKB200_ACT_NONE) {      // uniform over the grid
+                lo = gate_activation(qkv.activation, lo);
+                hi = gate_activation(qkv.activation, hi);
+              }
               __nv_bfloat162 pair = __floats2bfloat162_rn(lo, hi);
               ow[e] = *reinterpret_cast<unsigned*>(&pair);
             }
@@ -764,7 +768,7 @@ static int make_out_map(CUtensorMap* map, void* base, long long M, long long N, 
 template <int BLOCK_N, int STAGES, bool OUT_F32, bool GATED = false, bool QKV = false, bool PAIR = false>
 static int launch_tc_persistent(const void* x, const void* w, const float* bias, void* out, int M, int N,
                                 int K, cudaStream_t stream, int k_splits = 1,
-                                const QkvEpilogue* qkv_in = nullptr, int activation = TOKB200_ACT_SILU) {
+                                const QkvEpilogue* qkv_in = nullptr, int activation = TOKB200_ACT_NONE) {
   using S = TcPersistentSmem<BLOCK_N, STAGES, OUT_F32, GATED, PAIR>;
   static_assert(S::kTotal <= 227 * 1024, "shared memory of one CTA");
   CUtensorMap map_x, map_w, map_out;
@@ -853,7 +857,7 @@ TOKB200_API int tokb200_gemm_tcgen05_error(void) {
 }
 
 TOKB200_API int tokb200_gemm_tcgen05(const void* x, const void* w, const float* bias, void* out,
-                                     int out_is_f32, int M, int N, int K, int block_n,
+                                     int out_is_f32, int M, int N, int K, int block_n, int activation,
                                      cudaStream_t stream) {
   if (M <= 0 || N <= 0) return TOKB200_OK;
   if (K <= 0 || K % 8) return TOKB200_BAD_SIZE;          // TMA: row pitch a multiple of 16 bytes
@@ -862,15 +866,18 @@ TOKB200_API int tokb200_gemm_tcgen05(const void* x, const void* w, const float* 
   if (M > 128 * 65535) return TOKB200_BAD_SIZE;
   // block_n + 1000 asks for the persistent kernel (TMA-stored output): the output's
   // row pitch must then be a multiple of 16 bytes
+  if (activation != TOKB200_ACT_NONE &&                  // the persistent kernel's bfloat16 epilogue alone applies one
+      (block_n < 1000 || out_is_f32 || activation < 0 || activation >= TOKB200_ACT_COUNT))
+    return TOKB200_BAD_SIZE;
   if (block_n >= 1000) {
     if ((out_is_f32 ? N % 4 : N % 8) != 0) return TOKB200_BAD_SIZE;
     switch (block_n - 1000) {
       case 128:
         return out_is_f32 ? launch_tc_persistent<128, 4, true>(x, w, bias, out, M, N, K, stream)
-                          : launch_tc_persistent<128, 5, false>(x, w, bias, out, M, N, K, stream);
+                          : launch_tc_persistent<128, 5, false>(x, w, bias, out, M, N, K, stream, 1, nullptr, activation);
       case 256:
         return out_is_f32 ? TOKB200_BAD_SIZE
-                          : launch_tc_persistent<256, 3, false>(x, w, bias, out, M, N, K, stream);
+                          : launch_tc_persistent<256, 3, false>(x, w, bias, out, M, N, K, stream, 1, nullptr, activation);
       default: return TOKB200_BAD_SIZE;
     }
   }
@@ -900,12 +907,14 @@ TOKB200_API int tokb200_gemm_tcgen05_partials(const void* x, const void* w, void
 // The pair form (two CTAs a tile of 256 rows x 256 columns; see the kernel).  kind 0: out [M,N]
 // bfloat16 (+ bias); kind 1: the gated product, out [M, N/2] bfloat16 (N a multiple of 256, no
 // bias); kind 2: float32 partial sums out [k_splits, M, N] (no bias); kind 3: as kind 0 with
-// 128-column tiles.  `activation`: the gated product's activation tag (kind 1 only).
+// 128-column tiles.  `activation`: the gated product's activation tag (kind 1), or that of the whole product (kinds 0
+// and 3; TOKB200_ACT_NONE for none).
 TOKB200_API int tokb200_gemm_tcgen05_pair(const void* x, const void* w, const float* bias, void* out,
                                           int kind, int M, int N, int K, int k_splits, int activation,
                                           cudaStream_t stream) {
   if (M <= 0 || N <= 0) return TOKB200_OK;
-  if (K <= 0 || K % 8 || k_splits < 1 || activation < 0 || activation >= TOKB200_ACT_COUNT) return TOKB200_BAD_SIZE;
+  if (K <= 0 || K % 8 || k_splits < 1 || activation < (kind == 1 ? 0 : TOKB200_ACT_NONE) || activation >= TOKB200_ACT_COUNT)
+    return TOKB200_BAD_SIZE;
   if (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) return TOKB200_BAD_ALIGNMENT;
   if (M > 128 * 65535) return TOKB200_BAD_SIZE;
   const int k_blocks = (K + TC_BLOCK_K - 1) / TC_BLOCK_K;
@@ -914,7 +923,7 @@ TOKB200_API int tokb200_gemm_tcgen05_pair(const void* x, const void* w, const fl
   switch (kind) {
     case 0:
       if (N % 8 || k_splits != 1) return TOKB200_BAD_SIZE;
-      return launch_tc_persistent<256, 5, false, false, false, true>(x, w, bias, out, M, N, K, stream);
+      return launch_tc_persistent<256, 5, false, false, false, true>(x, w, bias, out, M, N, K, stream, 1, nullptr, activation);
     case 1:
       if (N % 256 || k_splits != 1 || bias) return TOKB200_BAD_SIZE;
       return launch_tc_persistent<256, 6, false, true, false, true>(x, w, nullptr, out, M, N, K, stream, 1,
@@ -924,7 +933,7 @@ TOKB200_API int tokb200_gemm_tcgen05_pair(const void* x, const void* w, const fl
       return launch_tc_persistent<256, 5, true, false, false, true>(x, w, nullptr, out, M, N, K, stream, k_splits);
     case 3:
       if (N % 8 || k_splits != 1) return TOKB200_BAD_SIZE;
-      return launch_tc_persistent<128, 6, false, false, false, true>(x, w, bias, out, M, N, K, stream);
+      return launch_tc_persistent<128, 6, false, false, false, true>(x, w, bias, out, M, N, K, stream, 1, nullptr, activation);
     default: return TOKB200_BAD_SIZE;
   }
 }

@@ -163,3 +163,214 @@ TOKB200_API int tokb200_rotate_interleaved(void* x, int dtype, int heads, int he
                             (__nv_bfloat16*)x, heads, head_row, lane0, dims, inv_freq, pos, row_req, n_rows);
   return TOKB200_BAD_DTYPE;
 }
+
+// ---- queries straight from the mixer's input, and values that pass a gate -------------------
+//
+// latent_rotate_store: one projection's output row holds the key/value latent with its positional key part (c_at ..)
+// and, for every head, a query in the cache row's own lanes (q_at .., `row` a head: kv_rank lanes without position,
+// rot_dim with, the rest zero).  The latent is RMS-normed with its gain, the positional parts of the key and of every
+// query are rotated (lane 2i with lane 2i + 1), the key row goes to the cache, the queries to q_out.  A block a token,
+// a warp a row; the angles are formed in 64-bit and brought into one turn before sine and cosine, once a token.
+template <typename TO>
+__global__ void __launch_bounds__(256)
+latent_rotate_store_kernel(const float* __restrict__ proj, int ld, int c_at, int q_at, int heads, int kv_rank, int rot_dim,
+                           int rot_dims, int row, const float* __restrict__ c_gain, float eps,
+                           const double* __restrict__ inv_freq, const int* __restrict__ pos,
+                           const int* __restrict__ row_req, const int* __restrict__ slot, TO* __restrict__ q_out,
+                           TO* __restrict__ pool) {
+  extern __shared__ float angles[];          // cosines, then sines, one a frequency
+  const int half = rot_dims >> 1;
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  const int r = row_req[t], p = pos[t];
+  const int where = slot ? slot[t] : -1;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    double a = (double)p * inv_freq[i];
+    a -= 6.283185307179586476925 * rint(a * 0.15915494309189533577);
+    float sn, cs;
+    sincosf((float)a, &sn, &cs);
+    angles[i] = cs;
+    angles[half + i] = sn;
+  }
+  pdl_wait();
+  pdl_launch();
+  if (r < 0) return;
+  __syncthreads();
+  const float* in = proj + (size_t)t * ld;
+  // lane l of a rotated part that starts at `part`
+  auto rotated = [&](const float* part, int l) {
+    const float own = part[l];
+    if (l >= rot_dims) return own;
+    const float other = part[l ^ 1], c = angles[l >> 1], s = angles[half + (l >> 1)];
+    return (l & 1) ? own * c + other * s : own * c - other * s;
+  };
+  for (int item = warp; item <= heads; item += warps) {
+    if (item == 0) {                          // the latent and the shared key part
+      if (where < 0) continue;
+      const float* c = in + c_at;
+      float squares = 0.f;
+      for (int l = lane; l < kv_rank; l += 32) squares = fmaf(c[l], c[l], squares);
+      const float inv = 1.0f / sqrtf(warp_sum(squares) / (float)kv_rank + eps);
+      TO* dst = pool + (size_t)where * row;
+      for (int l = lane; l < row; l += 32) {
+        float v = 0.f;
+        if (l < kv_rank) v = c[l] * inv * c_gain[l];
+        else if (l < kv_rank + rot_dim) v = rotated(c + kv_rank, l - kv_rank);
+        dst[l] = from_float<TO>(v);
+      }
+    } else {
+      const float* q = in + q_at + (size_t)(item - 1) * row;
+      TO* dst = q_out + ((size_t)t * heads + item - 1) * row;
+      for (int l = lane; l < row; l += 32)
+        dst[l] = from_float<TO>((l < kv_rank || l >= kv_rank + rot_dim) ? q[l] : rotated(q + kv_rank, l - kv_rank));
+    }
+  }
+}
+
+TOKB200_API int tokb200_latent_rotate_store(const float* proj, int ld, int c_at, int q_at, int heads, int kv_rank,
+                                            int rot_dim, int rot_dims, int row, const float* c_gain, float eps,
+                                            const double* inv_freq, const int* pos, const int* row_req, const int* slot,
+                                            void* q_out, void* pool, int out_dtype, int n_rows, cudaStream_t stream) {
+  if (n_rows <= 0) return TOKB200_OK;
+  if (heads <= 0 || kv_rank <= 0 || rot_dim < 0 || rot_dims < 0 || rot_dims > rot_dim || (rot_dims & 1) ||
+      row < kv_rank + rot_dim || c_at + kv_rank + rot_dim > ld || q_at + heads * row > ld || rot_dims > 8192 ||
+      (rot_dims > 0 && inv_freq == nullptr))
+    return TOKB200_BAD_SIZE;
+  const int warps = heads + 1 < 8 ? heads + 1 : 8;
+  const size_t smem = (size_t)rot_dims * sizeof(float);
+#define LAUNCH(TO)                                                                                                     \
+  return launch_dependent(latent_rotate_store_kernel<TO>, dim3(n_rows), dim3(warps * 32), smem, stream, proj, ld, c_at, \
+                          q_at, heads, kv_rank, rot_dim, rot_dims, row, c_gain, eps, inv_freq, pos, row_req, slot,      \
+                          (TO*)q_out, (TO*)pool)
+  if (out_dtype == TOKB200_F32) LAUNCH(float);
+  if (out_dtype == TOKB200_BF16) LAUNCH(__nv_bfloat16);
+#undef LAUNCH
+  return TOKB200_BAD_DTYPE;
+}
+
+// latent_values: the heads' values from their weighted latents, through a gate:
+//     out[t, h, l] = (sum_c w[h, l, c] mixed[t, h, c]) * sigmoid(gate[t, g_at + h vdim + l])
+// mixed [T, heads, row], w per head.  In bfloat16 (w [heads, vdim, row], row in whole 16s) a product on tensor cores
+// whose epilogue applies the gate: it is bound by reading mixed and gate, not by its arithmetic (row and vdim are a
+// hundred or so).  A tile is 64 lanes of a head by 64 rows (a warp 16 rows), or, with few rows, by 16 (a warp 16 lanes);
+// k goes through shared memory in pieces of 64.
+#define LV_K 64
+#define LV_PITCH (LV_K + 8)
+template <bool FEW>
+__global__ void __launch_bounds__(128)
+latent_values_mma_kernel(const __nv_bfloat16* __restrict__ mixed, const __nv_bfloat16* __restrict__ w,
+                         const float* __restrict__ gate, int ld, int g_at, int heads, int vdim, int row,
+                         __nv_bfloat16* __restrict__ out, int n_rows) {
+  constexpr int ROWS = FEW ? 16 : 64, TILES = FEW ? 2 : 8;      // TILES: pieces of 8 lanes a warp
+  __shared__ __align__(16) __nv_bfloat16 a_s[ROWS][LV_PITCH];
+  __shared__ __align__(16) __nv_bfloat16 w_s[64][LV_PITCH];
+  const int t0 = blockIdx.x * ROWS, head = blockIdx.y, l0 = blockIdx.z * 64;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int row_in = FEW ? 0 : warp * 16, lane_in = FEW ? warp * 16 : 0;
+  const __nv_bfloat16* wh = w + (size_t)head * vdim * row;
+  auto stage_w = [&](int k0) {
+    for (int i = threadIdx.x; i < 64 * (LV_K / 8); i += 128) {
+      const int l = i / (LV_K / 8), k = (i % (LV_K / 8)) * 8;
+      uint4 v = make_uint4(0u, 0u, 0u, 0u);
+      if (l0 + l < vdim && k0 + k < row) v = *reinterpret_cast<const uint4*>(wh + (size_t)(l0 + l) * row + k0 + k);
+      *reinterpret_cast<uint4*>(&w_s[l][k]) = v;
+    }
+  };
+  stage_w(0);                                 // weights are written by no kernel of the step
+  pdl_wait();
+  pdl_launch();
+  float acc[TILES][4];
+#pragma unroll
+  for (int j = 0; j < TILES; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+  for (int k0 = 0; k0 < row; k0 += LV_K) {
+    if (k0) {
+      __syncthreads();                        // the piece before has been read
+      stage_w(k0);
+    }
+    for (int i = threadIdx.x; i < ROWS * (LV_K / 8); i += 128) {
+      const int m = i / (LV_K / 8), k = (i % (LV_K / 8)) * 8;
+      uint4 v = make_uint4(0u, 0u, 0u, 0u);
+      if (t0 + m < n_rows && k0 + k < row)
+        v = *reinterpret_cast<const uint4*>(mixed + ((size_t)(t0 + m) * heads + head) * row + k0 + k);
+      *reinterpret_cast<uint4*>(&a_s[m][k]) = v;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < LV_K; k += 16) {
+      unsigned a[4];
+      const unsigned from = (unsigned)__cvta_generic_to_shared(&a_s[row_in + (lane & 15)][k + (lane >> 4) * 8]);
+      asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                   : "=r"(a[0]), "=r"(a[1]), "=r"(a[2]), "=r"(a[3]) : "r"(from));
+#pragma unroll
+      for (int j = 0; j < TILES; j += 2) {    // two pieces of 8 lanes a load
+        unsigned b[4];
+        const int l = lane_in + 8 * j + (lane & 7) + ((lane >> 4) << 3);
+        const unsigned at = (unsigned)__cvta_generic_to_shared(&w_s[l][k + ((lane >> 3) & 1) * 8]);
+        asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                     : "=r"(b[0]), "=r"(b[1]), "=r"(b[2]), "=r"(b[3]) : "r"(at));
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+          asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                       : "+f"(acc[j + h][0]), "+f"(acc[j + h][1]), "+f"(acc[j + h][2]), "+f"(acc[j + h][3])
+                       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[2 * h]), "r"(b[2 * h + 1]));
+      }
+    }
+  }
+  const int g = lane >> 2, q = lane & 3;
+#pragma unroll
+  for (int j = 0; j < TILES; ++j)
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int t = t0 + row_in + g + 8 * h, l = l0 + lane_in + 8 * j + 2 * q;
+      if (t >= n_rows || l >= vdim) continue;
+      const float* z = gate + (size_t)t * ld + g_at + head * vdim + l;
+      __nv_bfloat16* o = out + ((size_t)t * heads + head) * vdim + l;
+      const float v0 = acc[j][2 * h] / (1.0f + expf(-z[0]));
+      if ((vdim & 1) == 0) {
+        *reinterpret_cast<__nv_bfloat162*>(o) = __floats2bfloat162_rn(v0, acc[j][2 * h + 1] / (1.0f + expf(-z[1])));
+      } else {
+        o[0] = __float2bfloat16_rn(v0);
+        if (l + 1 < vdim) o[1] = __float2bfloat16_rn(acc[j][2 * h + 1] / (1.0f + expf(-z[1])));
+      }
+    }
+}
+
+// The 32-bit form (w [heads, row, vdim]: neighbouring threads on neighbouring lanes), k in index order: a block a
+// (row, head), the weighted latent in shared memory.
+__global__ void __launch_bounds__(128)
+latent_values_f32_kernel(const float* __restrict__ mixed, const float* __restrict__ w, const float* __restrict__ gate,
+                         int ld, int g_at, int heads, int vdim, int row, float* __restrict__ out) {
+  extern __shared__ float latent_s[];
+  const int t = blockIdx.x, head = blockIdx.y;
+  pdl_wait();
+  pdl_launch();
+  const float* in = mixed + ((size_t)t * heads + head) * row;
+  for (int c = threadIdx.x; c < row; c += blockDim.x) latent_s[c] = in[c];
+  __syncthreads();
+  const float* wh = w + (size_t)head * row * vdim;
+  for (int l = threadIdx.x; l < vdim; l += blockDim.x) {
+    float sum = 0.f;
+    for (int c = 0; c < row; ++c) sum = fmaf(wh[(size_t)c * vdim + l], latent_s[c], sum);
+    out[((size_t)t * heads + head) * vdim + l] = sum / (1.0f + expf(-gate[(size_t)t * ld + g_at + head * vdim + l]));
+  }
+}
+
+// w: [heads, vdim, row] in bfloat16, [heads, row, vdim] in float32.
+TOKB200_API int tokb200_latent_values(const void* mixed, const void* w, const float* gate, int ld, int g_at, int heads,
+                                      int vdim, int row, void* out, int dtype, int n_rows, cudaStream_t stream) {
+  if (n_rows <= 0) return TOKB200_OK;
+  if (heads <= 0 || heads > 65535 || vdim <= 0 || row <= 0 || row > 8192 || g_at + heads * vdim > ld) return TOKB200_BAD_SIZE;
+  if (dtype == TOKB200_F32)
+    return launch_dependent(latent_values_f32_kernel, dim3(n_rows, heads), dim3(vdim <= 32 ? 32 : vdim <= 64 ? 64 : 128),
+                            (size_t)row * sizeof(float), stream, (const float*)mixed, (const float*)w, gate, ld, g_at, heads,
+                            vdim, row, (float*)out);
+  if (dtype != TOKB200_BF16) return TOKB200_BAD_DTYPE;
+  if (row % 16 || (((uintptr_t)mixed | (uintptr_t)w) & 15) || ((uintptr_t)out & 3)) return TOKB200_BAD_ALIGNMENT;
+  const bool few = n_rows <= 64;
+  const dim3 grid((n_rows + (few ? 15 : 63)) / (few ? 16 : 64), heads, (vdim + 63) / 64);
+#define LAUNCH(FEW)                                                                                              \
+  return launch_dependent(latent_values_mma_kernel<FEW>, grid, dim3(128), 0, stream, (const __nv_bfloat16*)mixed, \
+                          (const __nv_bfloat16*)w, gate, ld, g_at, heads, vdim, row, (__nv_bfloat16*)out, n_rows)
+  if (few) LAUNCH(true);
+  LAUNCH(false);
+#undef LAUNCH
+}

@@ -221,6 +221,7 @@ linear_ring_kernel(const LrParams p) {
           reinterpret_cast<float*>(p.out)[((size_t)split * p.M + m) * p.N + n] = v;
         } else {
           if (p.bias) v += p.bias[n];
+          if (p.act != TOKB200_ACT_NONE) v = gate_activation(p.act, v);
           if (p.out_is_f32) reinterpret_cast<float*>(p.out)[(size_t)m * p.N + n] = v;
           else reinterpret_cast<__nv_bfloat16*>(p.out)[(size_t)m * p.N + n] = __float2bfloat16_rn(v);
         }
@@ -291,17 +292,19 @@ static int lr_launch(const LrParams& p, const LrPlan& plan, cudaStream_t stream)
 }
 
 // out: [M, N] bfloat16 or float32 when k_splits == 1 (bias added); float32 partial sums
-// [k_splits, M, N] otherwise (no bias: the consumer adds them up).
+// [k_splits, M, N] otherwise (no bias: the consumer adds them up).  `act`: the activation of a whole product,
+// TOKB200_ACT_NONE for none.
 TOKB200_API int tokb200_linear_ring(const void* x, const void* w, const float* bias, void* out, int out_is_f32,
-                                    int M, int N, int K, int k_splits, cudaStream_t stream) {
+                                    int M, int N, int K, int k_splits, int act, cudaStream_t stream) {
   const LrPlan plan = lr_plan(M, N, K, k_splits, false);
   if (plan.blocks == 0) return TOKB200_BAD_SIZE;
-  if (k_splits > 1 && (bias || !out_is_f32)) return TOKB200_BAD_SIZE;
+  if (k_splits > 1 && (bias || !out_is_f32 || act != TOKB200_ACT_NONE)) return TOKB200_BAD_SIZE;
+  if (act < TOKB200_ACT_NONE || act >= TOKB200_ACT_COUNT) return TOKB200_BAD_SIZE;
   if (((uintptr_t)x | (uintptr_t)w) & 15) return TOKB200_BAD_ALIGNMENT;
   LrParams p;
   p.x = (const __nv_bfloat16*)x; p.w = (const __nv_bfloat16*)w; p.bias = bias; p.out = out; p.out_is_f32 = out_is_f32;
   p.M = M; p.N = N; p.K = K; p.k_splits = k_splits; p.k_per_split = plan.k_per_split; p.depth = plan.depth;
-  p.x_pitch = plan.x_pitch; p.act = 0;
+  p.x_pitch = plan.x_pitch; p.act = act;
   return M <= 8 ? lr_launch<1, false>(p, plan, stream)
                 : M <= 16 ? lr_launch<2, false>(p, plan, stream) : lr_launch<4, false>(p, plan, stream);
 }

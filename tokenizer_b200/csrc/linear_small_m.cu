@@ -41,7 +41,8 @@ __device__ __forceinline__ uint4 load16(const __nv_bfloat16* p, bool ok) {
 // block's warps split into TPB teams of LSM_WARPS / TPB warps, a team per row tile.
 // GATED: w [N, K] holds, for every 128 outputs, their 128 "gate" rows followed by
 // their 128 "up" rows; a row tile is then 8 gate rows and the 8 up rows of the same
-// outputs, and the result is act(gate) * up, [M, N / 2] (`act`: the activation's tag).
+// outputs, and the result is act(gate) * up, [M, N / 2] (`act`: the activation's tag).  Not GATED and k not cut: the
+// result is act(product + bias), `act` TOKB200_ACT_NONE for the product as it is.
 // DENSE (9 to 16 rows, a weight of up to LSM_DENSE_ELEMENTS): the kernel is held to 80 registers so
 // that three blocks fit a multiprocessor.  A small matrix gains from the loads in flight (hidden
 // 896, 16 rows: 0.86 -> 0.80 ms a decoding step); a large one loses (3584 x 18944: 38 -> 55 us).
@@ -174,6 +175,7 @@ linear_small_m_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* 
       reinterpret_cast<float*>(out)[((size_t)blockIdx.y * M + m) * N + n] = v;
     } else {
       if (bias) v += bias[n];
+      if (act != TOKB200_ACT_NONE) v = gate_activation(act, v);
       if (out_is_f32) reinterpret_cast<float*>(out)[(size_t)m * N + n] = v;
       else reinterpret_cast<__nv_bfloat16*>(out)[(size_t)m * N + n] = __float2bfloat16_rn(v);
     }
@@ -210,7 +212,7 @@ static int launch_small_m_gated(const void* x, const void* w, void* out, int M, 
 
 template <int MT>
 static int launch_small_m(const void* x, const void* w, const float* bias, void* out,
-                          int out_is_f32, int M, int N, int K, int k_splits,
+                          int out_is_f32, int M, int N, int K, int k_splits, int act,
                           cudaStream_t stream) {
   const int tiles = (N + 15) / 16;
   int k_per_split = (K + k_splits - 1) / k_splits;
@@ -221,37 +223,39 @@ static int launch_small_m(const void* x, const void* w, const float* bias, void*
       if (tiles >= 1024)
         return launch_dependent(linear_small_m_kernel<MT, 2, false, true>, dim3((tiles + 1) / 2, k_splits),
                                 dim3(LSM_THREADS), 0, stream, (const __nv_bfloat16*)x, (const __nv_bfloat16*)w,
-                                bias, out, out_is_f32, M, N, K, k_per_split, 0);
+                                bias, out, out_is_f32, M, N, K, k_per_split, act);
       return launch_dependent(linear_small_m_kernel<MT, 1, false, true>, dim3(tiles, k_splits), dim3(LSM_THREADS),
                               0, stream, (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, bias, out, out_is_f32,
-                              M, N, K, k_per_split, 0);
+                              M, N, K, k_per_split, act);
     }
   }
   if (tiles >= 1024) {
     dim3 grid((tiles + 1) / 2, k_splits);
     return launch_dependent(linear_small_m_kernel<MT, 2, false>, grid, dim3(LSM_THREADS), 0, stream,
                             (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, bias, out, out_is_f32,
-                            M, N, K, k_per_split, 0);
+                            M, N, K, k_per_split, act);
   }
   dim3 grid(tiles, k_splits);
   return launch_dependent(linear_small_m_kernel<MT, 1, false>, grid, dim3(LSM_THREADS), 0, stream,
                           (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, bias, out, out_is_f32,
-                          M, N, K, k_per_split, 0);
+                          M, N, K, k_per_split, act);
 }
 
 // out: [M, N] bfloat16 or float32 when k_splits == 1 (bias added); float32
-// partial sums [k_splits, M, N] otherwise (no bias: the consumer adds them up).
+// partial sums [k_splits, M, N] otherwise (no bias: the consumer adds them up).  `act`: the activation of a whole
+// product, TOKB200_ACT_NONE for none.
 TOKB200_API int tokb200_linear_small_m(const void* x, const void* w, const float* bias, void* out,
-                                       int out_is_f32, int M, int N, int K, int k_splits,
+                                       int out_is_f32, int M, int N, int K, int k_splits, int act,
                                        cudaStream_t stream) {
   if (M <= 0 || N <= 0) return TOKB200_OK;
   if (M > 64 || K <= 0 || K % 8 || k_splits < 1 || k_splits > 64) return TOKB200_BAD_SIZE;
-  if (k_splits > 1 && (bias || !out_is_f32)) return TOKB200_BAD_SIZE;
+  if (k_splits > 1 && (bias || !out_is_f32 || act != TOKB200_ACT_NONE)) return TOKB200_BAD_SIZE;
+  if (act < TOKB200_ACT_NONE || act >= TOKB200_ACT_COUNT) return TOKB200_BAD_SIZE;
   if (((uintptr_t)x | (uintptr_t)w) & 15) return TOKB200_BAD_ALIGNMENT;
-  if (M <= 8) return launch_small_m<1>(x, w, bias, out, out_is_f32, M, N, K, k_splits, stream);
-  if (M <= 16) return launch_small_m<2>(x, w, bias, out, out_is_f32, M, N, K, k_splits, stream);
-  if (M <= 32) return launch_small_m<4>(x, w, bias, out, out_is_f32, M, N, K, k_splits, stream);
-  return launch_small_m<8>(x, w, bias, out, out_is_f32, M, N, K, k_splits, stream);
+  if (M <= 8) return launch_small_m<1>(x, w, bias, out, out_is_f32, M, N, K, k_splits, act, stream);
+  if (M <= 16) return launch_small_m<2>(x, w, bias, out, out_is_f32, M, N, K, k_splits, act, stream);
+  if (M <= 32) return launch_small_m<4>(x, w, bias, out, out_is_f32, M, N, K, k_splits, act, stream);
+  return launch_small_m<8>(x, w, bias, out, out_is_f32, M, N, K, k_splits, act, stream);
 }
 
 // out[M, N/2] (bfloat16) = act(x Wg^T) * (x Wu^T), w in the 128-gate / 128-up row

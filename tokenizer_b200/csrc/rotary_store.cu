@@ -24,6 +24,9 @@
 // cosines are computed once a frequency into shared memory (every head turns by the same angles).  `kv_heads` = 0: the
 // projection holds queries only (a layer that reads another layer's cache): nothing is written but q_out.
 //
+// `values_are_keys`: there are no v columns; a token's values are its keys as projected (bias added, before norms and
+// rotation), vdim = dim.
+//
 // attention_gate: out[t, h, l] *= sigmoid(proj[t, at + h * vdim + l]), l < vdim, on rows of `row` lanes a
 // head: a gate on the heads' outputs that is one more projection of the mixer's input.
 #include "common.cuh"
@@ -59,7 +62,7 @@ __global__ void qkv_rotate_store_kernel(const TI* __restrict__ proj, int ld, int
                                         T* __restrict__ k_pool, T* __restrict__ v_pool, int heads, int kv_heads,
                                         int dim, int vdim, int row, const float* __restrict__ q_gain,
                                         const float* __restrict__ k_gain, float eps, const float* __restrict__ temp,
-                                        int half_layout, int head_norm, float head_eps, int quads, float magnitude) {
+                                        int half_layout, int head_norm, float head_eps, int quads, float magnitude, int v_col) {
   // shared memory: a token's cosines and sines, one pair a frequency (every head turns by the same
   // angles), then the heads' inverse root mean squares (with `head_norm`)
   extern __shared__ float shared[];
@@ -189,7 +192,7 @@ __global__ void qkv_rotate_store_kernel(const TI* __restrict__ proj, int ld, int
       } else if (where >= 0) {
         const int g = head - heads - kv_heads;
         T* dst = v_pool + ((size_t)where * kv_heads + g) * row;
-        const int col0 = (heads + kv_heads) * dim + g * vdim;
+        const int col0 = v_col + g * vdim;
         for (int l = lane * 4; l < row; l += 128) {
           float v[4] = {0.f, 0.f, 0.f, 0.f};
           if (l < vdim) rs_load4(fin, col0 + l, bias, nullptr, 0, 1.f, v);
@@ -234,7 +237,7 @@ __global__ void qkv_rotate_store_kernel(const TI* __restrict__ proj, int ld, int
     } else if (where >= 0) {
       const int g = head - heads - kv_heads;
       T* dst = v_pool + ((size_t)where * kv_heads + g) * row;
-      const int col0 = (heads + kv_heads) * dim + g * vdim;
+      const int col0 = v_col + g * vdim;
       for (int l = lane; l < row; l += 32) {
         float value = 0.f;
         if (l < vdim) value = to_float(in[col0 + l]) + (bias ? bias[col0 + l] : 0.f);
@@ -251,9 +254,11 @@ TOKB200_API int tokb200_qkv_rotate_store(const void* proj, int proj_dtype, int l
                                          int out_dtype, int n_rows, int heads, int kv_heads, int dim, int vdim,
                                          int row, const float* q_gain, const float* k_gain, float eps,
                                          const float* temp, int half_layout, int head_norm, float head_eps,
-                                         float magnitude, cudaStream_t stream) {
+                                         float magnitude, int values_are_keys, cudaStream_t stream) {
   if (n_rows <= 0) return TOKB200_OK;
   if (kv_heads == 0 && (slot != nullptr || k_gain != nullptr)) return TOKB200_BAD_SIZE;
+  if (values_are_keys && (vdim != dim || kv_heads == 0)) return TOKB200_BAD_SIZE;
+  const int v_col = (values_are_keys ? heads : heads + kv_heads) * dim;      // the values' first column
   const size_t smem = (size_t)(rot_dims + (head_norm ? heads + kv_heads : 0)) * sizeof(float);
   if (smem > 40000) return TOKB200_BAD_SIZE;
   // four lanes a thread: float32 products whose columns, heads and rows are whole 4s (rotated lanes whole 8s, so
@@ -270,7 +275,7 @@ TOKB200_API int tokb200_qkv_rotate_store(const void* proj, int proj_dtype, int l
                           (const TI*)proj, ld, at, bias, inv_freq, inv_freq64, rot_dims, pos, slot, row_req,  \
                           (T*)q_out,                                                                          \
                           (T*)k_pool, (T*)v_pool, heads, kv_heads, dim, vdim, row, q_gain, k_gain, eps, temp, \
-                          half_layout, head_norm, head_eps, quads, magnitude)
+                          half_layout, head_norm, head_eps, quads, magnitude, v_col)
   if (proj_dtype == TOKB200_F32 && out_dtype == TOKB200_F32) LAUNCH(float, float);
   if (proj_dtype == TOKB200_F32 && out_dtype == TOKB200_BF16) LAUNCH(float, __nv_bfloat16);
   if (proj_dtype == TOKB200_BF16 && out_dtype == TOKB200_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);

@@ -285,8 +285,9 @@ def rope_store(qkv, bias, pos, slot, cos, sin, q_out, k_pool, v_pool, nh, nkv, d
         _stream()), "rope_store")
 
 
-# The activation of a gated feed-forward is a parameter of every kernel that applies one.
-ACTIVATIONS = {"silu": 0, "gelu_pytorch_tanh": 1, "relu": 2}
+# The activation of a feed-forward is a parameter of every kernel that applies one.
+ACTIVATIONS = {"silu": 0, "gelu_pytorch_tanh": 1, "relu": 2, "relu_squared": 3}
+NO_ACTIVATION = -1
 
 
 def activation_tag(name: str) -> int:
@@ -294,6 +295,21 @@ def activation_tag(name: str) -> int:
         return ACTIVATIONS[name]
     except KeyError:
         raise ValueError(f"the gated kernels know the activations {', '.join(ACTIVATIONS)}; found {name!r}") from None
+
+
+def product_activation(name: Optional[str]) -> int:
+    """The tag of the activation in a plain product's epilogue (None: the product as it is)."""
+    return NO_ACTIVATION if name is None else activation_tag(name)
+
+
+def activate(z: torch.Tensor, activation: str, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """out = act(z), element by element (`out` None: in place)."""
+    out = z if out is None else out
+    if out.shape != z.shape or out.dtype != z.dtype:
+        raise ValueError("activate: out has the shape and type of z")
+    _check(_lib("activation").tokb200_activate(
+        _ptr(z), _ptr(out), _i(_tag(z)), _i(activation_tag(activation)), _ll(z.numel()), _stream()), "activate")
+    return out
 
 
 def silu_gate(gu: torch.Tensor, out: torch.Tensor, activation: str = "silu") -> None:
@@ -520,8 +536,8 @@ def linear_small_m_supported(M: int, K: int) -> bool:
     return 0 < M <= 64 and K % 8 == 0
 
 
-def linear_small_m(x, w, bias, out, k_splits: int = 1) -> None:
-    """out = x w^T (+ bias) for at most 64 rows of bfloat16 x.  With k_splits > 1
+def linear_small_m(x, w, bias, out, k_splits: int = 1, activation: Optional[str] = None) -> None:
+    """out = act(x w^T (+ bias)) for at most 64 rows of bfloat16 x (`activation` None: no act).  With k_splits > 1
     `out` is float32 [k_splits, M, N]: partial sums that the consumer adds."""
     M, K = x.shape
     N = w.shape[0]
@@ -534,7 +550,7 @@ def linear_small_m(x, w, bias, out, k_splits: int = 1) -> None:
         raise ValueError(f"linear_small_m: out must be {want}")
     _check(_lib("linear_small_m").tokb200_linear_small_m(
         _ptr(x), _ptr(w), _ptr(bias), _ptr(out), _i(1 if out.dtype == torch.float32 else 0),
-        _i(M), _i(N), _i(K), _i(k_splits), _stream()), "linear_small_m")
+        _i(M), _i(N), _i(K), _i(k_splits), _i(product_activation(activation)), _stream()), "linear_small_m")
 
 
 PREFILL_TILE_ROWS = 64
@@ -581,9 +597,10 @@ def gemm_tcgen05_supported(M: int, N: int, K: int) -> bool:
     return M > 0 and N > 0 and K > 0 and K % 8 == 0
 
 
-def gemm_tcgen05(a, w, bias, out, block_n: int = 0) -> None:
+def gemm_tcgen05(a, w, bias, out, block_n: int = 0, activation: Optional[str] = None) -> None:
     """out[M,N] = a[M,K] w[N,K]^T (+ bias) on tcgen05 tensor cores with TMA-fed
-    operands; bfloat16 in, bfloat16 or float32 out.  K must be a multiple of 8."""
+    operands; bfloat16 in, bfloat16 or float32 out.  K must be a multiple of 8.  `activation` (bfloat16 out, N a
+    multiple of 8): applied in the persistent kernel's epilogue."""
     M, K = a.shape
     N = w.shape[0]
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or w.shape[1] != K:
@@ -594,7 +611,7 @@ def gemm_tcgen05(a, w, bias, out, block_n: int = 0) -> None:
         raise ValueError("gemm_tcgen05: out is [M,N] bfloat16 or float32")
     if not block_n:
         pitch_ok = N % (4 if out.dtype == torch.float32 else 8) == 0
-        if pitch_ok and M * N >= 128 * 128 * 32:
+        if pitch_ok and (M * N >= 128 * 128 * 32 or activation is not None):
             # persistent kernel, TMA-stored output: the wide tile where it divides the work well
             # (with one tile of rows, the narrow tile gives twice the blocks to stream the weights)
             block_n = 1256 if (out.dtype == torch.bfloat16 and N >= 2048 and M > 128) else 1128
@@ -602,7 +619,7 @@ def gemm_tcgen05(a, w, bias, out, block_n: int = 0) -> None:
             block_n = 128 if N > 64 else 64
     _check(_lib("gemm_tcgen05").tokb200_gemm_tcgen05(
         _ptr(a), _ptr(w), _ptr(bias), _ptr(out), _i(1 if out.dtype == torch.float32 else 0),
-        _i(M), _i(N), _i(K), _i(block_n), _stream()), "gemm_tcgen05")
+        _i(M), _i(N), _i(K), _i(block_n), _i(product_activation(activation)), _stream()), "gemm_tcgen05")
 
 
 def gemm_tcgen05_partials(a, w, out) -> None:
@@ -626,10 +643,10 @@ PAIR_PLAIN, PAIR_GATED, PAIR_PARTIALS, PAIR_PLAIN_128 = 0, 1, 2, 3
 _PAIR = os.environ.get("TOKB200_GEMM_PAIR", "1") != "0"
 
 
-def gemm_tcgen05_pair(a, w, bias, out, kind: int, activation: str = "silu") -> None:
+def gemm_tcgen05_pair(a, w, bias, out, kind: int, activation: Optional[str] = None) -> None:
     """The product on pairs of CTAs (two SMs a tile of 256 rows x 256 columns, each loading half
-    of the tile's rows of w).  PAIR_PLAIN: out [M,N] bfloat16 (+ bias); PAIR_GATED: out [M,N/2]
-    bfloat16 = silu(gate) * up for w from `interleave_gate_up`; PAIR_PARTIALS: out [S,M,N]
+    of the tile's rows of w).  PAIR_PLAIN: out [M,N] bfloat16 (+ bias, then the `activation` where one is named);
+    PAIR_GATED: out [M,N/2] bfloat16 = act(gate) * up (silu unless named) for w from `interleave_gate_up`; PAIR_PARTIALS: out [S,M,N]
     float32 partial sums over S pieces of k; PAIR_PLAIN_128: as PAIR_PLAIN with 128-column tiles."""
     M, K = a.shape
     N = w.shape[0]
@@ -652,7 +669,8 @@ def gemm_tcgen05_pair(a, w, bias, out, kind: int, activation: str = "silu") -> N
         raise ValueError("gemm_tcgen05_pair: K a multiple of 8, N of 8 (4 for partial sums)")
     _check(_lib("gemm_tcgen05").tokb200_gemm_tcgen05_pair(
         _ptr(a), _ptr(w), _ptr(bias), _ptr(out), _i(kind), _i(M), _i(N), _i(K), _i(splits),
-        _i(activation_tag(activation)), _stream()), "gemm_tcgen05_pair")
+        _i(activation_tag(activation or "silu") if kind == PAIR_GATED else product_activation(activation)), _stream()),
+        "gemm_tcgen05_pair")
 
 
 def gemm_tcgen05_check() -> None:
@@ -969,8 +987,8 @@ def linear_ring_splits(M: int, N: int, K: int, sms: int) -> int:
     return best
 
 
-def linear_ring(x, w, bias, out, k_splits: int = 1) -> None:
-    """out = x @ w.T (+ bias) for up to 16 rows and a large weight (bfloat16 in; out [M,N]
+def linear_ring(x, w, bias, out, k_splits: int = 1, activation: Optional[str] = None) -> None:
+    """out = act(x @ w.T (+ bias)) (`activation` None: no act) for up to 16 rows and a large weight (bfloat16 in; out [M,N]
     bfloat16/float32, or float32 partial sums [k_splits, M, N] without bias)."""
     M, K = x.shape
     N = w.shape[0]
@@ -985,7 +1003,7 @@ def linear_ring(x, w, bias, out, k_splits: int = 1) -> None:
         raise ValueError("linear_ring: out is [M,N] bfloat16 or float32")
     _check(_lib("linear_ring").tokb200_linear_ring(
         _ptr(x), _ptr(w), _ptr(bias), _ptr(out), _i(1 if out.dtype == torch.float32 else 0), _i(M), _i(N), _i(K),
-        _i(k_splits), _stream()), "linear_ring")
+        _i(k_splits), _i(product_activation(activation)), _stream()), "linear_ring")
 
 
 def linear_ring_gated(x, w, out, activation: str = "silu") -> None:
@@ -1372,7 +1390,7 @@ def stream_update(x: torch.Tensor, y=None, base=None, carried=None, share=None, 
 def qkv_rotate_store(proj: torch.Tensor, at: int, bias, inv_freq, rot_dims: int, pos, slot, row_req, q_out, k_pool,
                      v_pool, heads: int, kv_heads: int, dim: int, vdim: int, row: int, q_gain=None, k_gain=None,
                      eps: float = 0.0, temp=None, layout: str = "interleaved", head_norm_eps: Optional[float] = None,
-                     magnitude: float = 1.0) -> None:
+                     magnitude: float = 1.0, values_are_keys: bool = False) -> None:
     """Bias, interleaved rotation of the first `rot_dims` lanes of every query and key head, and the
     cache write, from `proj`'s columns at .. (q, k, v); rows of `row` lanes a head, zero behind dim
     (queries, keys) and vdim (values).  `slot` None: no cache write.  `q_gain` / `k_gain` (float32, one a
@@ -1382,15 +1400,18 @@ def qkv_rotate_store(proj: torch.Tensor, at: int, bias, inv_freq, rot_dims: int,
     `head_norm_eps` (a number): after the rotation every query and key head is divided by its own root mean
     square over its dim lanes, that eps inside the root.  `inv_freq` float64: the angle position * frequency is
     taken in 64-bit and brought into one turn before its sine and cosine (float32: the 32-bit product).  `magnitude` multiplies cosine and sine (1 with `head_norm_eps`).  `kv_heads` 0: `proj` holds queries only and nothing
-    but `q_out` is written (`slot`, `k_pool`, `v_pool` None)."""
+    but `q_out` is written (`slot`, `k_pool`, `v_pool` None).  `values_are_keys`: `proj` has no v columns; a
+    token's values are its keys as projected (bias added; no norm, no rotation), vdim = dim."""
     n = proj.shape[0]
+    if values_are_keys and (vdim != dim or kv_heads == 0):
+        raise ValueError("qkv_rotate_store: values that are the keys have the keys' lanes")
     if layout not in ("interleaved", "half"):
         raise ValueError("qkv_rotate_store: the rotated lanes pair interleaved or by halves")
     if kv_heads == 0 and (slot is not None or k_gain is not None):
         raise ValueError("qkv_rotate_store: a projection of queries alone writes no cache rows")
     if tuple(q_out.shape) != (n, heads * row) or \
             (kv_heads and (k_pool.dtype != q_out.dtype or v_pool.dtype != q_out.dtype)) or \
-            at + heads * dim + kv_heads * (dim + vdim) > proj.shape[1]:
+            at + heads * dim + kv_heads * (dim if values_are_keys else dim + vdim) > proj.shape[1]:
         raise ValueError("qkv_rotate_store: q_out is [T, heads * row] in the cache's type, the columns inside proj")
     for gain, size in ((q_gain, heads * dim), (k_gain, kv_heads * dim), (temp, heads)):
         if gain is not None and (gain.dtype != torch.float32 or gain.numel() != size):
@@ -1401,8 +1422,8 @@ def qkv_rotate_store(proj: torch.Tensor, at: int, bias, inv_freq, rot_dims: int,
         _ptr(inv_freq if wide else None), _i(rot_dims), _ptr(pos),
         _ptr(slot), _ptr(row_req), _ptr(q_out), _ptr(k_pool), _ptr(v_pool), _i(_tag(q_out)), _i(n), _i(heads),
         _i(kv_heads), _i(dim), _i(vdim), _i(row), _ptr(q_gain), _ptr(k_gain), _f(eps), _ptr(temp),
-        _i(int(layout == "half")), _i(int(head_norm_eps is not None)), _f(head_norm_eps or 0.0), _f(magnitude), _stream()),
-        "qkv_rotate_store")
+        _i(int(layout == "half")), _i(int(head_norm_eps is not None)), _f(head_norm_eps or 0.0), _f(magnitude),
+        _i(int(values_are_keys)), _stream()), "qkv_rotate_store")
 
 
 def attention_gate(out: torch.Tensor, proj: torch.Tensor, at: int, heads: int, vdim: int, row: int) -> None:
@@ -1600,6 +1621,144 @@ def mamba2_out_norm(y: torch.Tensor, proj: torch.Tensor, z_at: int, gain: torch.
     _check(_lib("mamba2").tokb200_mamba2_out_norm(
         _ptr(y), _sliced_ptr(proj), _i(_tag(proj)), _i(_ld(proj)), _i(z_at), _ptr(gain), _f(eps), _i(inner), _i(parts),
         _ptr(row_req), _ptr(out), _i(_tag(out)), _i(n), _stream()), "mamba2_out_norm")
+
+
+# ---- several residual streams ----
+STREAMS_MAX = 8
+
+
+def streams_step(x: torch.Tensor, streams: int, y=None, mix=None, share=None, read=None, gain=None, eps: float = 0.0,
+                 out: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x float32 [T, streams, H], or [T, H] where all streams are still equal.  With `y` ([T, H] or float32 partial sums
+    [S, T, H]): x_t <- sum_s mix[s, t] x_s + share[t] y, in place (a new tensor where the streams were equal); returns
+    the streams.  With `out` [T, H]: out = u, or u / sqrt(mean(u^2) + eps) * gain, u = sum_s read[s] x_s of the new
+    streams (`read` None: their sum).  `rows` (int32): only those rows are read, `out` is dense, x stays as it is.
+    mix [streams, streams] (from the row to the column), share and read [streams], gain [H]: float32."""
+    equal, hidden = x.dim() == 2, x.shape[-1]
+    n_rows = x.shape[0] if rows is None else rows.shape[0]
+    if x.dtype != torch.float32 or (not equal and (x.dim() != 3 or x.shape[1] != streams)) or not 1 <= streams <= STREAMS_MAX:
+        raise ValueError(f"streams_step: float32 [T, H] or [T, streams, H], 1 to {STREAMS_MAX} streams")
+    for v, size in ((mix, streams * streams), (share, streams), (read, streams), (gain, hidden)):
+        if v is not None and (v.dtype != torch.float32 or v.numel() != size):
+            raise ValueError("streams_step: the weights are float32, one a stream (or pair of streams), the gain one a lane")
+    if (y is not None and (mix is None or share is None)) or (out is not None and tuple(out.shape) != (n_rows, hidden)) or \
+            (out is None and (gain is not None or y is None)):
+        raise ValueError("streams_step: an output with its weights, a norm with its result [T, H]")
+    flat = x if equal else x[:, 0]
+    n_partials, stride = _partials(y, flat) if y is not None else (1, 0)
+    x_out = None
+    if y is not None and rows is None:
+        x_out = torch.empty((x.shape[0], streams, hidden), dtype=torch.float32, device=x.device) if equal else x
+    _check(_lib("streams").tokb200_streams_step(
+        _ptr(x), _i(int(equal)), _ptr(x_out), _i(streams), _ptr(y), _i(_tag(y) if y is not None else F32), _i(n_partials),
+        _ll(stride), _ptr(mix), _ptr(share), _ptr(read), _ptr(gain), _f(eps), _ptr(out),
+        _i(_tag(out) if out is not None else F32), _ptr(rows), _i(n_rows), _i(hidden), _stream()), "streams_step")
+    return x if x_out is None else x_out
+
+
+# ---- attention over a latent: queries straight from the mixer's input, gated values ----
+def latent_rotate_store(proj: torch.Tensor, c_at: int, q_at: int, heads: int, kv_rank: int, rot_dim: int, rot_dims: int,
+                        row: int, c_gain, eps: float, inv_freq, pos, row_req, slot, q_out, pool) -> None:
+    """From a float32 product's rows: the normed latent and the rotated positional key part into the token's cache row
+    (`pool` [slots, 1, row]), and every head's query (columns q_at .., `row` a head) with its positional lanes rotated
+    into `q_out` [T, heads * row].  `inv_freq` float64; `slot` None: no cache write."""
+    n = proj.shape[0]
+    if proj.dtype != torch.float32 or tuple(q_out.shape) != (n, heads * row) or pool.dtype != q_out.dtype or \
+            pool.shape[-1] * pool.shape[-2] != row or q_at + heads * row > proj.shape[1] or \
+            (inv_freq is not None and inv_freq.dtype != torch.float64):
+        raise ValueError("latent_rotate_store: a float32 product, queries and pool of `row` lanes in one type, 64-bit frequencies")
+    _check(_lib("latent").tokb200_latent_rotate_store(
+        _sliced_ptr(proj), _i(_ld(proj)), _i(c_at), _i(q_at), _i(heads), _i(kv_rank), _i(rot_dim), _i(rot_dims), _i(row),
+        _ptr(c_gain), _f(eps), _ptr(inv_freq), _ptr(pos), _ptr(row_req), _ptr(slot), _ptr(q_out), _ptr(pool), _i(_tag(pool)),
+        _i(n), _stream()), "latent_rotate_store")
+
+
+def latent_values(mixed: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, g_at: int, heads: int, vdim: int, row: int,
+                  out: torch.Tensor) -> None:
+    """out[t, h] = (w[h] mixed[t, h]) * sigmoid(gate[t, g_at + h vdim ..]); `mixed` [T, heads * row], `out` [T, heads *
+    vdim], `gate` a float32 product; w [heads, vdim, row] in bfloat16 (row in whole 16s), [heads, row, vdim] in float32."""
+    n = mixed.shape[0]
+    shape = (heads, vdim, row) if mixed.dtype == torch.bfloat16 else (heads, row, vdim)
+    if tuple(mixed.shape) != (n, heads * row) or tuple(out.shape) != (n, heads * vdim) or tuple(w.shape) != shape or \
+            w.dtype != mixed.dtype or out.dtype != mixed.dtype or gate.dtype != torch.float32 or gate.shape[0] != n or \
+            g_at + heads * vdim > gate.shape[1]:
+        raise ValueError("latent_values: sizes or types of the latents, the weights, the gate or the output disagree")
+    _check(_lib("latent").tokb200_latent_values(
+        _ptr(mixed), _ptr(w), _sliced_ptr(gate), _i(_ld(gate)), _i(g_at), _i(heads), _i(vdim), _i(row), _ptr(out),
+        _i(_tag(out)), _i(n), _stream()), "latent_values")
+
+
+# ---- the matrix memory with exponential gates ----
+MLSTM_MAX_DIM = 256
+
+
+def mlstm_gates(proj: torch.Tensor, i_at: int, f_at: int, i_bias, f_bias, cap: float, heads: int, state: torch.Tensor,
+                m_off: int, q_start, state_slot, gates: torch.Tensor) -> None:
+    """The running maximum of every request's rows (`state` [slots, n]: it starts from and ends in the heads' numbers at
+    m_off), and `gates` float32 [3, heads, >= T]: what a token's matrix is kept by, what its write is weighed by, and
+    exp(-maximum)."""
+    if proj.dtype != torch.float32 or gates.dtype != torch.float32 or gates.shape[:2] != (3, heads) or \
+            state.dtype != torch.float32 or state.dim() != 2 or \
+            any(v.dtype != torch.float32 or v.numel() != heads for v in (i_bias, f_bias)):
+        raise ValueError("mlstm_gates: a float32 product, biases one a head, gates [3, heads, T]")
+    _check(_lib("mlstm").tokb200_mlstm_gates(
+        _sliced_ptr(proj), _i(_ld(proj)), _i(i_at), _i(f_at), _ptr(i_bias), _ptr(f_bias), _f(cap), _i(heads), _ptr(state),
+        _ll(state.shape[1]), _i(m_off), _ptr(q_start), _ptr(state_slot), _i(q_start.shape[0] - 1), _i(proj.shape[0]),
+        _ptr(gates[0]), _ptr(gates[1]), _ptr(gates[2]), _ll(gates.shape[2]), _stream()), "mlstm_gates")
+
+
+def mlstm_scan(proj: torch.Tensor, q_at: int, k_at: int, v_at: int, heads: int, dim: int, vdim: int, gates: torch.Tensor,
+               state: torch.Tensor, q_start, state_slot, y: torch.Tensor, yn: torch.Tensor,
+               segments: Optional[int] = None) -> None:
+    """S <- keep S + add k v^T, n <- keep n + add k; y [T, heads * vdim] = S^T q dim^(-1/2), yn [T, heads] = n . q
+    dim^(-1/2), over every request's rows; a slot of `state` starts with [heads, vdim + 1, dim] (n behind the columns).
+    `segments` as for `mamba2_scan`."""
+    n = proj.shape[0]
+    if proj.dtype != torch.float32 or y.dtype != torch.float32 or tuple(y.shape) != (n, heads * vdim) or \
+            tuple(yn.shape) != (n, heads) or yn.dtype != torch.float32 or gates.shape[:2] != (3, heads) or gates.shape[2] < n or \
+            state.dtype != torch.float32 or state.dim() != 2 or heads * (vdim + 1) * dim > state.shape[1]:
+        raise ValueError("mlstm_scan: sizes of the product, the gates, the state or the outputs disagree")
+    n_requests = q_start.shape[0] - 1
+    if segments is None:
+        segments = mamba2_segments(n, n_requests, heads, vdim)
+    if not 1 <= segments <= MAMBA2_MAX_SEGMENTS:
+        raise ValueError(f"mlstm_scan: 1 to {MAMBA2_MAX_SEGMENTS} segments")
+    scratch = torch.empty(n_requests * segments * heads * ((vdim + 1) * dim + 1), dtype=torch.float32,
+                          device=proj.device) if segments > 1 else None
+    _check(_lib("mlstm").tokb200_mlstm_scan(
+        _sliced_ptr(proj), _i(_ld(proj)), _i(q_at), _i(k_at), _i(v_at), _i(heads), _i(dim), _i(vdim), _f(dim ** -0.5),
+        _ptr(gates[0]), _ptr(gates[1]), _ll(gates.shape[2]), _ptr(state), _ll(state.shape[1]), _ptr(q_start), _ptr(state_slot),
+        _i(n_requests), _ptr(y), _ptr(yn), _ptr(scratch), _i(segments), _stream()), "mlstm_scan")
+    if segments > 1:
+        counter.launches += 1
+
+
+def mlstm_out_norm(y: torch.Tensor, yn: torch.Tensor, gates: torch.Tensor, proj: torch.Tensor, g_at: int, gain, eps: float,
+                   heads: int, vdim: int, row_req, out: torch.Tensor) -> None:
+    """o = y / (max(|yn|, exp(-maximum)) + 1e-6), divided by its root mean square over vdim, times `gain` (one a lane of
+    all heads) and sigmoid(proj[:, g_at ..])."""
+    n = y.shape[0]
+    if tuple(out.shape) != (n, heads * vdim) or gain.numel() != heads * vdim or g_at + heads * vdim > proj.shape[1] or \
+            proj.dtype != torch.float32 or gates.shape[2] < n:
+        raise ValueError("mlstm_out_norm: sizes of the gain, the gate or the output disagree")
+    _check(_lib("mlstm").tokb200_mlstm_out_norm(
+        _ptr(y), _ptr(yn), _ptr(gates[2]), _ll(gates.shape[2]), _sliced_ptr(proj), _i(_ld(proj)), _i(g_at), _ptr(gain), _f(eps),
+        _i(heads), _i(vdim), _ptr(row_req), _ptr(out), _i(_tag(out)), _i(n), _stream()), "mlstm_out_norm")
+
+
+def mlstm_step(proj: torch.Tensor, q_at: int, k_at: int, v_at: int, g_at: int, i_at: int, f_at: int, i_bias, f_bias,
+               cap: float, heads: int, dim: int, vdim: int, gain, eps: float, state: torch.Tensor, m_off: int, row_req,
+               state_slot, out: torch.Tensor) -> None:
+    """A step in which every request brings ONE token: gates, recurrence, norm and gate in one kernel, a block a (row,
+    head)."""
+    n = proj.shape[0]
+    if proj.dtype != torch.float32 or tuple(out.shape) != (n, heads * vdim) or gain.numel() != heads * vdim or \
+            state.dtype != torch.float32 or state.dim() != 2 or m_off < heads * (vdim + 1) * dim:
+        raise ValueError("mlstm_step: sizes of the product, the state, the gain or the output disagree")
+    _check(_lib("mlstm").tokb200_mlstm_step(
+        _sliced_ptr(proj), _i(_ld(proj)), _i(q_at), _i(k_at), _i(v_at), _i(g_at), _i(i_at), _i(f_at), _ptr(i_bias), _ptr(f_bias),
+        _f(cap), _i(heads), _i(dim), _i(vdim), _f(dim ** -0.5), _ptr(gain), _f(eps), _ptr(state), _ll(state.shape[1]), _i(m_off),
+        _ptr(row_req), _ptr(state_slot), _i(n), _ptr(out), _i(_tag(out)), _stream()), "mlstm_step")
 
 
 # ---- read-only streams in the decoding kernels' access patterns (bench.py --stream-probe) ----

@@ -28,6 +28,8 @@ def all_variants():
         ("moe.cu", (), ()),
         ("short_conv.cu", (), ()),
         ("mamba2.cu", (), ()),
+        ("mlstm.cu", (), ()),
+        ("streams.cu", (), ()),
     ]
     for head_dim in (16, 32, 48, 64, 128):
         jobs.append(("attention_decode.cu", (f"HEAD_DIM={head_dim}",), ()))

@@ -389,7 +389,8 @@ class RotaryGQAttention(PagedAttention):
     counts as softcap * tanh(s / softcap)); `output_gate` (the heads' outputs are multiplied by sigmoid(Wg h),
     tensor `.g`, heads * vdim rows; the product rides in the stacked input product); `unit_sink` (one added to
     the softmax's denominator: a sink of score 0 for every head, no tensor); `keep_first` (the sequence's first
-    keys that every query sees although its window or chunk has passed them); `own_kv` False (the layer
+    keys that every query sees although its window or chunk has passed them); `values_are_keys` (no v tensor: a
+    token's values are its keys as projected, bias added and not rotated; vdim = dim); `own_kv` False (the layer
     has no k and v tensors and is called on an earlier call's cache: it projects, rotates and norms queries
     only); `cache_chunk` (what the cache manager may give back, where other calls read this cache with chunks of
     their own: a chunk size that all of theirs divide, or None to keep every page)."""
@@ -398,15 +399,19 @@ class RotaryGQAttention(PagedAttention):
     def tensors(spec):
         p, x = spec.params, spec.prefix
         hidden, heads, groups, dim, vdim = p["hidden_size"], p["heads"], p["kv_heads"], p["dim"], p["vdim"]
-        own = p.get("own_kv", True)
+        own, values = p.get("own_kv", True), not p.get("values_are_keys")
         out = [TensorSpec(x + ".q", (heads * dim, hidden))]
         if own:
-            out += [TensorSpec(x + ".k", (groups * dim, hidden)), TensorSpec(x + ".v", (groups * vdim, hidden))]
+            out.append(TensorSpec(x + ".k", (groups * dim, hidden)))
+            if values:
+                out.append(TensorSpec(x + ".v", (groups * vdim, hidden)))
         out.append(TensorSpec(x + ".o", (hidden, heads * vdim)))
         if p.get("bias", True):
             out.append(TensorSpec(x + ".q.b", (heads * dim,)))
             if own:
-                out += [TensorSpec(x + ".k.b", (groups * dim,)), TensorSpec(x + ".v.b", (groups * vdim,))]
+                out.append(TensorSpec(x + ".k.b", (groups * dim,)))
+                if values:
+                    out.append(TensorSpec(x + ".v.b", (groups * vdim,)))
         if p.get("qk_norm"):
             out.append(TensorSpec(x + ".q.norm", (heads * dim,), "one_plus_normal", 0.1))
             if own:
@@ -430,6 +435,9 @@ class RotaryGQAttention(PagedAttention):
         self.keep_first = int(p.get("keep_first") or 0)
         self.softcap = float(p["softcap"]) if p.get("softcap") is not None else None
         self.own_kv = bool(p.get("own_kv", True))
+        self.values_are_keys = bool(p.get("values_are_keys"))
+        if self.values_are_keys and (self.vdim != self.dim or not self.own_kv):
+            raise ConfigError("values that are the layer's keys have the keys' lanes")
         self.cache_chunk = p["cache_chunk"] if "cache_chunk" in p else self.chunk
         self.head_norm = bool(p.get("head_norm"))
         if self.softcap is not None and self.softcap <= 0:
@@ -446,7 +454,7 @@ class RotaryGQAttention(PagedAttention):
             self.rot_dims = int(self.position.dims)
             if self.rot_dims > self.dim:
                 raise ConfigError(f"{self.rot_dims} rotated lanes do not fit a head of {self.dim}")
-        names = "qkv" if self.own_kv else "q"
+        names = "q" if not self.own_kv else "qk" if self.values_are_keys else "qkv"
         self._stack = [store.get(x + "." + n) for n in names]
         # the gate's pre-activations are more columns of the stacked product, behind q, k and v
         self.gate_at = None
@@ -501,7 +509,8 @@ class RotaryGQAttention(PagedAttention):
                              q_gain=self.q_gain, k_gain=self.k_gain, eps=self.norm_eps, temp=self.temp,
                              layout=getattr(self.position, "layout", "interleaved"),
                              magnitude=getattr(self.position, "magnitude", 1.0),
-                             head_norm_eps=self.norm_eps if self.head_norm else None)
+                             head_norm_eps=self.norm_eps if self.head_norm else None,
+                             values_are_keys=self.values_are_keys)
         mixed = self.runtime.empty(ctx.n_tokens, self.nh * self.row)
         self.attend(q, mixed, ctx, group, cache)
         if self.gate_at is not None:

@@ -34,6 +34,8 @@ Interfaces (duck-typed; the classes below marked "interface" document them):
   filter        tensors(spec); __init__(spec, store, runtime); state_need() -> StateNeed | None;
                 forward(h [T,H], ctx, state) -> what a sublayer reads instead of h (it may keep
                 its last inputs per request in `state`, the arena of the call's side state)
+  connection    tensors(spec); __init__(spec, store, runtime); read, mix, share (float32): how a sublayer is
+                connected to several residual streams (`StreamBundle`)
   scale         tensors(spec); __init__(spec, store, runtime); vector (float32 [H]): a learned
                 scale, element by element, on a sublayer's output before it is added
 """
@@ -48,7 +50,7 @@ from ..config.spec import ConfigError, PartSpec
 from ..kernels import ops
 
 CATEGORIES = ("mixer", "feed_forward", "norm", "position", "block", "embedding", "head", "gate", "injection",
-              "filter", "scale")
+              "filter", "scale", "connection")
 _REGISTRY: Dict[str, Dict[str, Any]] = {c: {} for c in CATEGORIES}
 
 
@@ -350,6 +352,15 @@ class ResidualStream:
         self.flush()
         self._gated = delta
 
+    def finish(self, norm, rows: torch.Tensor, runtime) -> torch.Tensor:
+        """The final norm of the wanted rows, everything pending added."""
+        self.flush()
+        return norm.forward(self.x, rows=rows)
+
+    def drop(self) -> None:
+        """Nobody reads the stream any more: what is pending is not added."""
+        self.pending = None
+
     def flush(self) -> torch.Tensor:
         pending = self.pending
         if pending is not None:
@@ -380,6 +391,63 @@ class ResidualStream:
             return fused(self.x, gated)
         delta, self.pending = self.pending, None
         return norm.forward(self.x, delta=delta)
+
+
+class StreamBundle:
+    """Several residual streams, float32 [T, streams, H], for arrangements whose sublayers read a weighted sum of the
+    streams and add to each of them (a `connection` part holds the weights).  The streams start equal and are kept as
+    one [T, H] until the first sublayer's output is added.  An output stays pending with its connection until the next
+    sublayer reads: mixing, adding, the weighted sum and the norm are then one kernel."""
+
+    def __init__(self, x: torch.Tensor, streams: int):
+        if x.dtype != torch.float32:
+            raise ValueError("the residual streams are float32")
+        self.x, self.streams = x, int(streams)
+        self._pending = None                      # (a sublayer's output, its connection)
+
+    def _step(self, **kw) -> None:
+        (y, link), self._pending = self._pending or (None, None), None
+        self.x = ops.streams_step(self.x, self.streams, y, link.mix if link is not None else None,
+                                  link.share if link is not None else None, **kw)
+
+    def read(self, norm, link, runtime) -> torch.Tensor:
+        """norm(sum of the streams, weighed by `link.read`), what is pending added first."""
+        fold = getattr(norm, "folded", None)
+        if fold is None:                          # a norm of another kind reads the weighted sum
+            u = torch.empty((self.x.shape[0], self.x.shape[-1]), dtype=torch.float32, device=self.x.device)
+            self._step(read=link.read, out=u)
+            return norm.forward(u)
+        gain, eps = fold()
+        h = runtime.empty(self.x.shape[0], self.x.shape[-1])
+        self._step(read=link.read, gain=gain, eps=eps, out=h)
+        return h
+
+    def add(self, y: torch.Tensor, link) -> None:
+        """Every stream anew from all of them and the output y: stays pending."""
+        if self._pending is not None:
+            self._step()
+        self._pending = (y, link)
+
+    def flush(self) -> torch.Tensor:
+        """The sum of the streams, float32 [T, H], everything pending added."""
+        if self._pending is not None:
+            self._step()
+        u = torch.empty((self.x.shape[0], self.x.shape[-1]), dtype=torch.float32, device=self.x.device)
+        self._step(out=u)
+        return u
+
+    def finish(self, norm, rows: torch.Tensor, runtime) -> torch.Tensor:
+        """norm(sum of the streams) of the wanted rows alone, what is pending counted in."""
+        fold = getattr(norm, "folded", None)
+        if fold is None:
+            return norm.forward(self.flush(), rows=rows)
+        gain, eps = fold()
+        h = runtime.empty(rows.shape[0], self.x.shape[-1])
+        self._step(gain=gain, eps=eps, out=h, rows=rows)
+        return h
+
+    def drop(self) -> None:
+        self._pending = None
 
 
 def build_part(category: str, spec: PartSpec, store, runtime: Runtime):

@@ -5,6 +5,7 @@ from __future__ import annotations
 
 import torch
 
+from ..config.spec import ConfigError
 from ..kernels import ops
 from ..weights.store import TensorSpec
 from .base import GatedDelta, StreamUpdate, register_part
@@ -332,3 +333,62 @@ register_part("scale", "layer_scale", LayerScale)
 register_part("filter", "causal_conv_residual", CausalConvResidual)
 register_part("block", "parallel_residual", ParallelResidual)
 register_part("block", "parallel_residual_mixer_only", ParallelResidualMixerOnly)
+
+
+class StreamConnection:
+    """How a sublayer is connected to the model's residual streams x_1 .. x_n: it reads sum_s in[s] x_s, and its output y
+    goes back as x_t <- sum_s mix[s, t] x_s + mult * out[t] * y, all streams at once from the old ones.  Tensors
+    `<prefix>.in` [n], `.out` [n], `.mix` [n, n]; `mult` (optional): a constant, taken into `.out` in float32."""
+
+    @staticmethod
+    def tensors(spec):
+        n, x = spec.params["streams"], spec.prefix
+        return [TensorSpec(x + ".in", (n,), "one_plus_normal", 0.1), TensorSpec(x + ".out", (n,), "one_plus_normal", 0.1),
+                TensorSpec(x + ".mix", (n, n), "normal", 0.5)]
+
+    def __init__(self, spec, store, runtime):
+        n, x = int(spec.params["streams"]), spec.prefix
+        if not 1 <= n <= ops.STREAMS_MAX:
+            raise ConfigError(f"a model has 1 to {ops.STREAMS_MAX} residual streams, found {n}")
+        self.runtime = runtime
+        self.read = runtime.vector(store.get(x + ".in"))
+        self.share = (runtime.vector(store.get(x + ".out")) * float(spec.params.get("mult", 1.0))).contiguous()
+        self.mix = runtime.vector(store.get(x + ".mix"))
+
+
+class ConnectedStreams:
+    """A pre-norm layer on several residual streams (`StreamBundle`): mixer and feed-forward each read the norm of a
+    weighted sum of the streams and add to all of them, by a `connection` of their own."""
+
+    PARTS = {"mixer": "mixer", "mixer_norm": "norm", "mixer_connection": "connection",
+             "feed_forward": "feed_forward", "feed_forward_norm": "norm", "feed_forward_connection": "connection"}
+
+    def __init__(self, mixer, mixer_norm, mixer_connection, feed_forward=None, feed_forward_norm=None,
+                 feed_forward_connection=None):
+        self.mixer, self.mixer_norm, self.mixer_connection = mixer, mixer_norm, mixer_connection
+        self.feed_forward, self.feed_forward_norm = feed_forward, feed_forward_norm
+        self.feed_forward_connection = feed_forward_connection
+
+    def streamed_weights(self):
+        out = []
+        for part in (self.mixer, self.feed_forward):
+            out += list(getattr(part, "streamed_weights", lambda: [])())
+        return out
+
+    def forward(self, streams, ctx, cache):
+        link = self.mixer_connection
+        streams.add(self.mixer.forward(streams.read(self.mixer_norm, link, link.runtime), ctx, cache), link)
+        if self.feed_forward is not None:
+            link = self.feed_forward_connection
+            streams.add(self.feed_forward.forward(streams.read(self.feed_forward_norm, link, link.runtime)), link)
+
+
+class ConnectedStreamsMixerOnly(ConnectedStreams):
+    """The same arrangement for a layer without a feed-forward."""
+
+    PARTS = {"mixer": "mixer", "mixer_norm": "norm", "mixer_connection": "connection"}
+
+
+register_part("connection", "stream_connection", StreamConnection)
+register_part("block", "connected_streams", ConnectedStreams)
+register_part("block", "connected_streams_mixer_only", ConnectedStreamsMixerOnly)

@@ -264,6 +264,32 @@ class RoutedMLP:
         return StreamUpdate(out, carried=h, share=share[:, columns - 1]) if self.identity else out
 
 
+class DenseMLP:
+    """Feed-forward without a gate: down(act(up(h))), no biases (tensors `<prefix>.up`, `.down`).  The activation is a
+    parameter (one of `ops.ACTIVATIONS`); in bfloat16 it is applied in the up product's epilogue, on the 32-bit sums."""
+
+    @staticmethod
+    def tensors(spec):
+        p, x = spec.params, spec.prefix
+        return [TensorSpec(x + ".up", (p["inner_size"], p["hidden_size"])),
+                TensorSpec(x + ".down", (p["hidden_size"], p["inner_size"]))]
+
+    def __init__(self, spec, store, runtime):
+        p, x = spec.params, spec.prefix
+        if p["activation"] not in ops.ACTIVATIONS:
+            raise ConfigError(f"dense feed-forward knows the activations {', '.join(ops.ACTIVATIONS)}; found {p['activation']}")
+        self.activation = p["activation"]
+        self.up = Linear(runtime.matrix(store.get(x + ".up")))
+        self.down = Linear(runtime.matrix(store.get(x + ".down")))
+
+    def streamed_weights(self):
+        return [self.up.weight, self.down.weight]
+
+    def forward(self, h):
+        return self.down.forward(self.up.forward(h, activation=self.activation), partials_ok=True)
+
+
+register_part("feed_forward", "dense_mlp", DenseMLP)
 register_part("feed_forward", "gated_mlp", GatedMLP)
 register_part("feed_forward", "routed_mlp", RoutedMLP)
 register_part("feed_forward", "poly_norm_mlp", PolyNormMLP)

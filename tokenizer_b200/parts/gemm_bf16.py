@@ -184,3 +184,27 @@ def linear_bf16(a: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tens
     if bias is not None:
         out.add_(bias.to(out.dtype) if out.dtype != torch.float32 else bias)
     return out
+
+
+def linear_bf16_activated(a: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], activation: str) -> torch.Tensor:
+    """act(a[M,K] weight[N,K]^T (+ bias)) as bfloat16 [M,N]: the activation in the epilogue of whichever kernel of the
+    framework the row count selects, on the 32-bit sums; where the vendor library's product leads (65 to LIBRARY_ROWS - 1
+    rows) or no such kernel takes the sizes, a kernel of its own behind the product."""
+    M, K = a.shape
+    N = weight.shape[0]
+    out = torch.empty((M, N), dtype=torch.bfloat16, device=a.device)
+    if ops._RING and M <= ops.RING_MAX_ROWS and (N * K >= ops.RING_ELEMENTS or M > ops.SMALL_M_ROWS) and \
+            ops.linear_ring_supported(M, N, K, 1):
+        ops.linear_ring(a, weight, bias, out, 1, activation)
+        return out
+    if ops.linear_small_m_supported(M, K) and (M <= ops.SMALL_M_ROWS or N < 4096):
+        ops.linear_small_m(a, weight, bias, out, 1, activation)
+        return out
+    if ops.gemm_tcgen05_supported(M, N, K) and N % 8 == 0 and os.environ.get("TOKB200_GEMM", "") != "library":
+        if ops._PAIR and M >= LIBRARY_ROWS:
+            ops.gemm_tcgen05_pair(a, weight, bias, out, ops.PAIR_PLAIN, activation)
+            return out
+        if M <= 64 or M >= LIBRARY_ROWS or os.environ.get("TOKB200_GEMM", "") == "own":
+            ops.gemm_tcgen05(a, weight, bias, out, activation=activation)
+            return out
+    return ops.activate(linear_bf16(a, weight, bias, torch.bfloat16), activation)

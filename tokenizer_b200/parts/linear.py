@@ -23,9 +23,10 @@ class Linear:
         self.out_features, self.in_features = weight.shape
 
     def forward(self, a: torch.Tensor, out_dtype: Optional[torch.dtype] = None,
-                use_bias: bool = True, partials_ok: bool = False) -> torch.Tensor:
+                use_bias: bool = True, partials_ok: bool = False, activation: Optional[str] = None) -> torch.Tensor:
         """[M, out] in `out_dtype` (default: the operands' type).  A caller whose
-        consumer adds partial sums (`partials_ok`) may get float32 [S, M, out]."""
+        consumer adds partial sums (`partials_ok`) may get float32 [S, M, out].  `activation` (one of
+        `ops.ACTIVATIONS`, not with `partials_ok`): applied to the result, in the product's epilogue where it has one."""
         if a.shape[-1] != self.in_features or a.dtype != self.weight.dtype:
             raise ValueError(
                 f"projection takes [{self.in_features}] rows of {self.weight.dtype}, "
@@ -37,5 +38,9 @@ class Linear:
         if a.dtype == torch.float32:
             out = torch.empty((a.shape[0], self.out_features), dtype=out_dtype, device=a.device)
             ops.gemm_f32(a, self.weight, bias, out)
-            return out
+            return out if activation is None else ops.activate(out, activation)
+        if activation is not None:
+            if partials_ok or out_dtype != torch.bfloat16:
+                raise ValueError("an activation comes with a whole product in the operands' type")
+            return gemm_bf16.linear_bf16_activated(a, self.weight, bias, activation)
         return gemm_bf16.linear_bf16(a, self.weight, bias, out_dtype, partials_ok)

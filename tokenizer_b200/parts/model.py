@@ -10,7 +10,7 @@ import torch
 from ..config.spec import ConfigError, ModelSpec
 from ..kernels import ops
 from ..weights.store import TensorSpec, WeightStore
-from .base import CacheBinding, ResidualStream, Runtime, StepContext, build_part, part_class
+from .base import CacheBinding, ResidualStream, Runtime, StepContext, StreamBundle, build_part, part_class
 
 
 def layer_parts(layer):
@@ -162,9 +162,10 @@ class DecoderModel:
 
     def _forward(self, ctx, bindings, want_rows):
         if getattr(self.embedding, "wants_positions", False):
-            stream = ResidualStream(self.embedding.forward(ctx.ids, ctx.pos, ctx.row_req))
+            x = self.embedding.forward(ctx.ids, ctx.pos, ctx.row_req)
         else:
-            stream = ResidualStream(self.embedding.forward(ctx.ids))
+            x = self.embedding.forward(ctx.ids)
+        stream = ResidualStream(x) if self.spec.streams is None else StreamBundle(x, self.spec.streams)
         # norms add in place: a part that adds the embedding's output again later gets a copy
         embedded = stream.x.clone() if self._keep_embedding else None
         ahead = self._prefetcher(ctx)
@@ -178,8 +179,6 @@ class DecoderModel:
         if ahead is not None:
             ahead.join()
         if want_rows.shape[0] == 0:
-            stream.pending = None
+            stream.drop()
             return torch.empty((0, self.vocab_size), dtype=torch.float32, device=self.runtime.device)
-        stream.flush()
-        h = self.final_norm.forward(stream.x, rows=want_rows)
-        return self.head.forward(h)
+        return self.head.forward(stream.finish(self.final_norm, want_rows, self.runtime))

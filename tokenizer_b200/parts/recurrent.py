@@ -1,5 +1,6 @@
 """Recurrent mixers: minGRU, the gated delta rule (`GatedDeltaNet`, below), the delta rule with a decay a
-key channel (`ChannelDeltaNet`) and the state-space recurrence (`Mamba2`).
+key channel (`ChannelDeltaNet`), the state-space recurrence (`Mamba2`) and the matrix memory with exponential gates
+(`MatrixMemory`).
 
 minGRU: a gated recurrence whose gates read only the current token.
 
@@ -414,7 +415,86 @@ class Mamba2:
         return self.out.forward(gated, partials_ok=True)
 
 
+class MatrixMemory:
+    """A matrix memory with exponential gates (the mLSTM).  From the mixer's input h: q = Wq h dim^(-1/2), k = Wk h (heads x
+    dim), v = Wv h (heads x vdim); per head the logarithms of two gates, each squashed into (-cap, cap) by a tanh:
+        i = cap tanh((Wi h + b_i) / cap),   f = log sigmoid(cap tanh((Wf h + b_f) / cap));
+    a matrix S, a vector n and a running maximum m, all zero at a sequence's start:
+        m' = max(f + m, i);  S <- exp(f + m - m') S + exp(i - m') k v^T;  n likewise with k alone;
+        o = S^T q / (max(|n . q|, exp(-m')) + 1e-6).
+    Every head's o is divided by its root mean square over vdim; the heads side by side, times the gain `.norm` (a lane of
+    all heads each) and sigmoid(Wg h), go through `.o`.  Tensors `<prefix>.q`, `.k`, `.v`, `.g`, `.i` (+ `.b`), `.f` (+
+    `.b`), `.norm`, `.o`.
+
+    The stacked input product is written in float32; everything behind it but the output projection's operand is 32-bit
+    (`csrc/mlstm.cu`).  Per request it keeps, in one state slot: the heads' matrices with n behind their columns
+    ([heads, vdim + 1, dim]), then the running maxima."""
+
+    graph_safe = True    # launches depend on device-side metadata alone
+
+    @staticmethod
+    def tensors(spec):
+        p, x = spec.params, spec.prefix
+        hidden, heads, dim, vdim = p["hidden_size"], p["heads"], p["dim"], p["vdim"]
+        return [TensorSpec(x + ".q", (heads * dim, hidden)), TensorSpec(x + ".k", (heads * dim, hidden)),
+                TensorSpec(x + ".v", (heads * vdim, hidden)), TensorSpec(x + ".g", (heads * vdim, hidden)),
+                TensorSpec(x + ".i", (heads, hidden)), TensorSpec(x + ".i.b", (heads,), "normal", 0.5),
+                TensorSpec(x + ".f", (heads, hidden)), TensorSpec(x + ".f.b", (heads,), "normal", 0.5),
+                TensorSpec(x + ".norm", (heads * vdim,), "one_plus_normal"), TensorSpec(x + ".o", (hidden, heads * vdim))]
+
+    def __init__(self, spec, store, runtime):
+        p, x = spec.params, spec.prefix
+        self.runtime = runtime
+        self.heads, self.dim, self.vdim = int(p["heads"]), int(p["dim"]), int(p["vdim"])
+        self.cap, self.eps = float(p["gate_cap"]), float(p["eps"])
+        if self.cap <= 0:
+            raise ConfigError("a cap on the gates is positive")
+        if not 1 <= self.dim <= ops.MLSTM_MAX_DIM:
+            raise ConfigError(f"the matrix memory takes heads of up to {ops.MLSTM_MAX_DIM} lanes; found {self.dim}")
+        names = ("q", "k", "v", "g", "i", "f")
+        weights = [store.get(x + "." + n) for n in names]
+        self.at, here = {}, 0
+        for name, w in zip(names, weights):
+            self.at[name], here = here, here + w.shape[0]
+        self.inputs = Linear(runtime.matrix(stacked_rows(weights)))
+        self.i_bias, self.f_bias = runtime.vector(store.get(x + ".i.b")), runtime.vector(store.get(x + ".f.b"))
+        self.gain = runtime.vector(store.get(x + ".norm"))
+        self.out = Linear(runtime.matrix(store.get(x + ".o")))
+        self.m_off = self.heads * (self.vdim + 1) * self.dim
+        self.state_floats = -(-(self.m_off + self.heads) // 4) * 4
+
+    def cache_need(self):
+        return CacheNeed(state=StateNeed((self.state_floats,)))
+
+    def shape_key(self, q_lens):
+        return "memory1" if max(q_lens) == 1 else "memory"      # the kernels' choice
+
+    def streamed_weights(self):
+        return [self.inputs.weight, self.out.weight]
+
+    def forward(self, h, ctx, cache):
+        n, heads, at = ctx.n_tokens, self.heads, self.at
+        proj = self.inputs.forward(h, out_dtype=torch.float32)
+        y = self.runtime.empty(n, heads * self.vdim)
+        if ctx.max_q_len == 1:
+            # every request brings one token: one kernel behind the input product
+            ops.mlstm_step(proj, at["q"], at["k"], at["v"], at["g"], at["i"], at["f"], self.i_bias, self.f_bias, self.cap,
+                           heads, self.dim, self.vdim, self.gain, self.eps, cache.state, self.m_off, ctx.row_req,
+                           ctx.state_slot, y)
+            return self.out.forward(y, partials_ok=True)
+        gates = torch.empty((3, heads, n), dtype=torch.float32, device=proj.device)
+        ops.mlstm_gates(proj, at["i"], at["f"], self.i_bias, self.f_bias, self.cap, heads, cache.state, self.m_off,
+                        ctx.q_start, ctx.state_slot, gates)
+        raw = torch.empty((n, heads * self.vdim), dtype=torch.float32, device=proj.device)
+        norm = torch.empty((n, heads), dtype=torch.float32, device=proj.device)
+        ops.mlstm_scan(proj, at["q"], at["k"], at["v"], heads, self.dim, self.vdim, gates, cache.state, ctx.q_start,
+                       ctx.state_slot, raw, norm)
+        ops.mlstm_out_norm(raw, norm, gates, proj, at["g"], self.gain, self.eps, heads, self.vdim, ctx.row_req, y)
+        return self.out.forward(y, partials_ok=True)
+
+
 register_part("mixer", "mamba2", Mamba2)
+register_part("mixer", "matrix_memory", MatrixMemory)
 register_part("mixer", "min_gru", MinGRU)
 register_part("mixer", "gated_delta_net", GatedDeltaNet)
 register_part("mixer", "channel_delta_net", ChannelDeltaNet)
