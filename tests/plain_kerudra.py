@@ -188,7 +188,7 @@ def forward(cfg, w, ids, keep=None):
     """Logits [T, vocab] of a whole sequence from its start.  `keep` (a list) receives the streams' sum after every
     layer run."""
     eps, m = float(cfg["norm"]["eps"]), float(cfg.get("residual_mult", 1.0))
-    x = w["embed"][torch.tensor(list(ids), dtype=torch.long)] * float(cfg["embedding"]["scale"])
+    x = w["embed"][torch.tensor(list(ids), dtype=torch.long)] * float((cfg.get("embedding") or {}).get("scale", 1.0))
     xs = torch.stack([x] * int(cfg["streams"]))
     for index in run_order(cfg):
         layer, p = cfg["layers"][index], f"l{index}."

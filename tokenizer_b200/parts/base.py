@@ -437,7 +437,8 @@ class StreamBundle:
         return u
 
     def finish(self, norm, rows: torch.Tensor, runtime) -> torch.Tensor:
-        """norm(sum of the streams) of the wanted rows alone, what is pending counted in."""
+        """norm(sum of the streams) of the wanted rows alone, what is pending counted in: the last thing a bundle does
+        (the streams themselves are not brought up to date)."""
         fold = getattr(norm, "folded", None)
         if fold is None:
             return norm.forward(self.flush(), rows=rows)
