@@ -3,7 +3,7 @@
 weights on one B200.  Prints ONE JSON line.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--impl ours|reference]
-                    [--config 0.5b|1.5b-mixed|7b|pufuzen|katopel|vizonex|zobelorn|kazepel]
+                    [--config 0.5b|1.5b-mixed|7b|pufuzen|katopel|vizonex|zobelorn|kazepel|kerudra]
 
 A "step" is one decode step of the whole batch.  `value` is decoded tokens a
 second timed on the device over K steps that never return to the host
@@ -197,14 +197,15 @@ def main():
     parser.add_argument("--layers", type=int, default=SIZES["num_hidden_layers"])
     parser.add_argument("--impl", default="ours", choices=["ours", "reference"])
     parser.add_argument("--config", default="0.5b", choices=["0.5b", "1.5b-mixed", "7b", "pufuzen", "katopel", "vizonex", "zobelorn",
-                                                           "kazepel"],
+                                                           "kazepel", "kerudra"],
                         help="0.5b: the headline line; 7b: the same at Qwen2.5-7B sizes with 8,192-token "
                              "contexts; 1.5b-mixed: 32 requests through the scheduler at Qwen2.5-1.5B sizes; "
                              "pufuzen: prefill and decoding of the Pufuzen design at two widths beside Qwen2 at "
                              "equal width, depth and parameters, and its kernels alone; katopel: the same for the Katopel design; "
                              "vizonex: the Vizonex design beside the Katopel design at equal width, depth and parameters; "
                              "zobelorn: the Zobelorn design beside Qwen2 at equal width, depth, heads and parameters; "
-                             "kazepel: the Kazepel design beside the Katopel design at equal width, depth and parameters")
+                             "kazepel: the Kazepel design beside the Katopel design at equal width, depth and parameters; "
+                             "kerudra: the Kerudra design beside the Pufuzen design at equal width, depth and parameters")
     parser.add_argument("--context", type=int, default=8192, help="--config 7b: tokens held before decoding")
     parser.add_argument("--layer-phases", action="store_true",
                         help="print where the time of the whole-layer kernel (TOKB200_LAYER=fused) goes, phase by "
@@ -219,7 +220,7 @@ def main():
     parser.add_argument("--only-decode", action="store_true",
                         help="time the decode steps only and print a short line (for profiling)")
     parser.add_argument("--only-kernels", action="store_true",
-                        help="--config katopel, vizonex, zobelorn, kazepel: the kernels alone, without the models")
+                        help="--config katopel, vizonex, zobelorn, kazepel, kerudra: the kernels alone, without the models")
     parser.add_argument("--only-prefill", action="store_true",
                         help="time the 2,048-token prefill only and print a short line (for profiling)")
     args = parser.parse_args()
@@ -251,6 +252,8 @@ def main():
         return run_zobelorn(args)
     if args.config == "kazepel":
         return run_kazepel(args)
+    if args.config == "kerudra":
+        return run_kerudra(args)
     args.steps = max(1, min(args.steps, NEW_TOKENS - args.warmup - 1))
 
     import torch
@@ -1783,6 +1786,213 @@ def run_kazepel(args):
         "unit": "tokens/s", "n_gpus": 1, "steps": steps, "warmup": args.warmup, "dtype": "bf16",
         "data": "synthetic: random weights drawn on the device, uniform random token ids",
         "config": {"sizes": KAZEPEL_SIZES, "prefill_tokens": PREFILL_TOKENS, "decode_context": context,
+                   "peaks": pk["source"], "hbm_gbs": pk["hbm_gbs"],
+                   "l2": "kernels alone: inputs larger than L2 and a 256 MB write between timed launches"},
+        "models": models, "kernels": kernels}))
+    return 0
+
+
+# ---- the Kerudra design beside the Pufuzen design at equal width, depth and parameter count ----
+KERUDRA_SIZES = {
+    # width, residual streams; latent attention of `heads` heads (dim unrotated and rot_dim rotated lanes, values of vdim,
+    # a latent of kv_rank, a window of `window` keys); attention of `heads` over `kv_heads` heads of dim lanes, half of them
+    # rotated; the matrix memory (m_heads matrices of m_dim x m_vdim).  The feed-forward's width is chosen so that the
+    # model has the parameters of the Pufuzen model of the same name.
+    "1k": dict(width=1024, streams=4, heads=16, kv_heads=4, dim=64, vdim=64, rot_dim=32, kv_rank=96, window=1024, m_heads=8,
+               m_dim=64, m_vdim=128, vocab=32000, layers=8),
+    "2k": dict(width=2048, streams=4, heads=16, kv_heads=4, dim=128, vdim=128, rot_dim=32, kv_rank=96, window=1024, m_heads=16,
+               m_dim=128, m_vdim=128, vocab=32000, layers=8),
+}
+
+
+def kerudra_config(z, ff, loop=None, streams=None):
+    """Latent attention, attention and the matrix memory in turn, every layer with a feed-forward."""
+    import tokenizer_b200 as tb
+    dense = {"kind": "dense", "ff": ff}
+    kinds = [
+        {"type": "latent_attention", "mlp": dense, "mixer": {
+            "heads": z["heads"], "dim": z["dim"], "rot_dim": z["rot_dim"], "vdim": z["vdim"], "kv_rank": z["kv_rank"],
+            "scale": (z["dim"] + z["rot_dim"]) ** -0.5, "mask": {"size": z["window"]}, "rot": {"base": 50000.0, "dims": z["rot_dim"]}}},
+        {"type": "attention", "mlp": dense, "mixer": {
+            "heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+            "rot": {"base": 500000.0, "dims": z["dim"] // 2}}},
+        {"type": "mlstm", "mlp": dense, "mixer": {"heads": z["m_heads"], "dim": z["m_dim"], "vdim": z["m_vdim"], "gate_cap": 15.0}}]
+    raw = {"architecture": "Kerudra", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "streams": streams or z["streams"],
+           "residual_mult": 0.8, "embedding": {"scale": 8.0}, "logit_scale": 0.5, "layers": [kinds[i % 3] for i in range(z["layers"])]}
+    if loop is not None:
+        raw["loop"] = dict(zip(("start", "stop", "times"), loop))
+    return tb.config.KerudraConfig.from_dict(raw)
+
+
+def run_kerudra(args):
+    """Prefill (one step of 2,048 tokens) and decoding (batch 1 and `--batch`, 2,048-token contexts) of the Kerudra
+    design at two widths, beside the closest design that was there, Pufuzen (latent attention, a recurrence, a dense
+    feed-forward), at the same width, depth and parameters, once more with two streams, and with four of its layers looped
+    twice; then the design's own kernels alone beside the like kernels of the other paths, each on inputs larger than
+    L2, against the measured copy peak."""
+    import torch
+    from tokenizer_b200.kernels import ops
+    from tokenizer_b200.parts import gemm_bf16
+    from tokenizer_b200.parts.model import declared_tensors
+
+    torch.cuda.set_device(0)
+    pk = peaks()
+    gen = torch.Generator().manual_seed(99)
+    context, steps = 2048, max(8, min(args.steps, 64))
+    timed = device_timed
+    count = lambda config: sum(int(torch.tensor(t.shape).prod()) for t in declared_tensors(config.model_spec()))
+
+    models = {}
+    for name, z in KERUDRA_SIZES.items():
+        if args.only_kernels:
+            break
+        beside = pufuzen_config(PUFUZEN_SIZES[name])
+        base, step = count(kerudra_config(z, 128)), count(kerudra_config(z, 256)) - count(kerudra_config(z, 128))
+        ff = max(1, round((count(beside) - base) / step) + 1) * 128
+        measure = lambda config: measure_design(config, z["vocab"], args, gen, context, steps)
+        models[name] = {"kerudra": dict(measure(kerudra_config(z, ff)), ff=ff), "pufuzen": measure(beside),
+                        "kerudra, two streams": measure(kerudra_config(z, ff, streams=2)),
+                        "kerudra, layers 2 .. 5 twice": measure(kerudra_config(z, ff, (2, 6, 2)))}
+
+    # ---- kernels alone: inputs larger than L2, a 256 MB write between the timed launches ----
+    dev = "cuda:0"
+    flush = torch.empty(64 << 20, dtype=torch.float32, device=dev)
+
+    def kernel_time(fn, reps=7):
+        times = []
+        for _ in range(3 + reps):
+            flush.zero_()
+            ms, _ = timed(fn)
+            times.append(ms)
+        return sorted(times[3:])[reps // 2]
+
+    kernels = {}
+
+    def record(name, ms, nbytes, like, flops=None):
+        kernels[name] = {"us": round(ms * 1e3, 1), "gb_s": round(nbytes / (ms / 1e3) / 1e9), "like": like,
+                         "of_measured_copy_peak": round(nbytes / (ms / 1e3) / 1e9 / pk["hbm_gbs"], 2)}
+        if flops is not None:
+            kernels[name]["tflops"] = round(flops / (ms / 1e3) / 1e12, 1)
+
+    ints = lambda values: torch.tensor(list(values), dtype=torch.int32, device=dev)
+    rnd = lambda *shape, dtype=torch.float32: torch.randn(*shape, device=dev, dtype=torch.float32).to(dtype)
+    bf16 = torch.bfloat16
+    T, H, rows = 8192, 2048, 64
+    # ---- the streams ----
+    y, h16, g1 = rnd(T, H, dtype=bf16), torch.empty(T, H, dtype=bf16, device=dev), torch.ones(H, device=dev)
+    for n in (2, 4):
+        x, mix, share, read = rnd(T, n, H), torch.eye(n, device=dev), torch.full((n,), 0.1, device=dev), torch.full((n,), 0.5, device=dev)
+        record(f"streams_step, {n} streams with a pending output and the norm, {T} x {H}",
+               kernel_time(lambda: ops.streams_step(x, n, y, mix, share, read=read, gain=g1, eps=1e-6, out=h16)),
+               T * H * (2 + 8 * n + 2), "rms_norm with pending add")
+    x = rnd(T, H)
+    record(f"rms_norm with pending add (Qwen2 path), {T} x {H}", kernel_time(lambda: ops.rms_norm(x, g1, 1e-6, h16, delta=y)),
+           T * H * (4 + 4 + 2 + 2), None)
+    del x, y
+    # ---- the matrix memory, beside the state-space recurrence with as many matrix elements ----
+    heads, dim, vdim = 16, 128, 128
+    at = dict(q=0, k=heads * dim, v=2 * heads * dim, g=2 * heads * dim + heads * vdim)
+    at["i"] = at["g"] + heads * vdim
+    proj = rnd(T, at["i"] + 2 * heads)
+    ib, fb, gain = torch.zeros(heads, device=dev), torch.full((heads,), 3.0, device=dev), torch.ones(heads * vdim, device=dev)
+    m_off = heads * (vdim + 1) * dim
+    slot = -(-(m_off + heads) // 4) * 4
+    y32, yn, gates = torch.empty(T, heads * vdim, device=dev), torch.empty(T, heads, device=dev), torch.empty(3, heads, T, device=dev)
+    y16 = torch.empty(T, heads * vdim, dtype=bf16, device=dev)
+    s_heads, s_vdim, n_state, groups = 32, 64, 128, 8
+    xbc, s_proj = rnd(T, s_heads * s_vdim + 2 * groups * n_state), rnd(T, s_heads)
+    zeros, ones = torch.zeros(s_heads, device=dev), torch.ones(s_heads, device=dev)
+    s_y = torch.empty(T, s_heads * s_vdim, device=dev)
+    for requests in (1, 4):
+        spans, slots = ints(T * r // requests for r in range(requests + 1)), ints(range(requests))
+        state, where = torch.zeros(requests, slot, device=dev), f"{T} tokens of {requests} request(s)"
+        record(f"mlstm_gates, {where}, {heads} heads",
+               kernel_time(lambda: ops.mlstm_gates(proj, at["i"], at["i"] + heads, ib, fb, 15.0, heads, state, m_off, spans, slots, gates)),
+               T * heads * 20, "gdn_prepare")
+        record(f"mlstm_scan, {where}, {heads} heads of {dim} x {vdim}",
+               kernel_time(lambda: ops.mlstm_scan(proj, at["q"], at["k"], at["v"], heads, dim, vdim, gates, state, spans, slots, y32, yn)),
+               T * heads * (2 * dim + 2 * vdim) * 4, "mamba2_scan", flops=T * heads * dim * (vdim + 1) * 6)
+        s_state = torch.zeros(requests, s_heads * s_vdim * n_state, device=dev)
+        record(f"mamba2_scan (Vizonex path), {where}, {s_heads} heads of {n_state} x {s_vdim}",
+               kernel_time(lambda: ops.mamba2_scan(xbc, s_proj, 0, zeros, zeros, ones, s_heads, groups, s_vdim, n_state, s_state, spans, slots, s_y)),
+               T * (2 * s_heads * s_vdim + 2 * groups * n_state) * 4, None, flops=T * s_heads * s_vdim * n_state * 6)
+    req0 = ints([0] * T)
+    record(f"mlstm_out_norm, {T} tokens x {heads} heads of {vdim}",
+           kernel_time(lambda: ops.mlstm_out_norm(y32, yn, gates, proj, at["g"], gain, 1e-6, heads, vdim, req0, y16)),
+           T * heads * vdim * (4 + 4 + 2), "gdn_out_norm")
+    gain_v = torch.ones(vdim, device=dev)
+    record(f"gdn_out_norm with a sigmoid gate (Kazepel path), {T} tokens x {heads} heads of {vdim}",
+           kernel_time(lambda: ops.gdn_out_norm(y32, proj, at["g"], gain_v, 1.0, 1e-6, y16, heads, vdim, req0, gate_kind="sigmoid")),
+           T * heads * vdim * (4 + 4 + 2), None)
+    spans, slots = ints(range(rows + 1)), ints(range(rows))
+    state = torch.zeros(rows, slot, device=dev)
+    record(f"mlstm_step, {rows} requests of one token, {heads} heads of {dim} x {vdim}",
+           kernel_time(lambda: ops.mlstm_step(proj[:rows], at["q"], at["k"], at["v"], at["g"], at["i"], at["i"] + heads, ib, fb, 15.0, heads,
+                                              dim, vdim, gain, 1e-6, state, m_off, slots, slots, y16[:rows])), rows * m_off * 8, "mamba2_scan, gdn_step")
+    s_state = torch.zeros(rows, s_heads * s_vdim * n_state, device=dev)
+    record(f"mamba2_scan (Vizonex path), {rows} requests of one token, {s_heads} heads of {n_state} x {s_vdim}",
+           kernel_time(lambda: ops.mamba2_scan(xbc[:rows], s_proj[:rows], 0, zeros, zeros, ones, s_heads, groups, s_vdim, n_state, s_state,
+                                               spans, slots, s_y[:rows])), rows * s_heads * s_vdim * n_state * 8, None)
+    del state, s_state, xbc, s_proj, s_y, y32
+    # ---- the latent: queries, cache row, gated values ----
+    nh, rank, rot, row, q_rank = 16, 96, 32, 128, 768
+    c_at, q_at, g_at = 0, rank + rot, rank + rot + nh * row
+    wide = rnd(T, g_at + nh * vdim)
+    freq64 = torch.tensor([5e4 ** (-2.0 * i / rot) for i in range(rot // 2)], dtype=torch.float64, device=dev)
+    freq32 = freq64.float()
+    pos, c_gain = torch.arange(T, dtype=torch.int32, device=dev), torch.ones(rank, device=dev)
+    q, pool = torch.empty(T, nh * row, dtype=bf16, device=dev), torch.zeros(T, 1, row, dtype=bf16, device=dev)
+    record(f"latent_rotate_store, {T} tokens, {nh} heads of {row} lanes",
+           kernel_time(lambda: ops.latent_rotate_store(wide, c_at, q_at, nh, rank, rot, rot, row, c_gain, 1e-6, freq64, pos, req0, pos, q, pool)),
+           T * (rank + rot + nh * row) * (4 + 2), "qkv_rotate_store, latent_prepare")
+    narrow, cq, q_gain = rnd(T, q_rank + rank + rot + H), torch.empty(T, q_rank, dtype=bf16, device=dev), torch.ones(q_rank, device=dev)
+    record(f"latent_prepare (Pufuzen path), {T} tokens, a query latent of {q_rank}",
+           kernel_time(lambda: ops.latent_prepare(narrow, 0, q_rank, q_rank, rank, rot, rot, q_gain, c_gain, 1e-6, freq32, pos, req0, pos, cq, pool)),
+           T * (q_rank + rank + rot) * (4 + 2), None)
+    del narrow
+    mixed, out = rnd(T, nh * row, dtype=bf16), torch.empty(T, nh * vdim, dtype=bf16, device=dev)
+    w_v = rnd(nh, vdim, row, dtype=bf16)
+    record(f"latent_values, {T} tokens, {nh} heads of {row} x {vdim}",
+           kernel_time(lambda: ops.latent_values(mixed, w_v, wide, g_at, nh, vdim, row, out)), T * nh * (row * 2 + vdim * 6), "attention_gate",
+           flops=T * nh * row * vdim * 2)
+    record(f"attention_gate (Zobelorn path), {T} tokens, {nh} heads of {vdim}",
+           kernel_time(lambda: ops.attention_gate(mixed, wide, g_at, nh, vdim, row)), T * nh * (row * 4 + vdim * 4), None)
+    del mixed, wide, w_v
+    # ---- attention whose values are its keys ----
+    nkv, d = 4, 128
+    wide = rnd(T, (nh + 2 * nkv) * d)
+    bias = torch.zeros((nh + 2 * nkv) * d, device=dev)
+    freq = torch.tensor([5e5 ** (-2.0 * i / 64) for i in range(32)], dtype=torch.float64, device=dev)
+    pools = [torch.zeros(T, nkv, d, dtype=bf16, device=dev) for _ in range(2)]
+    for shared in (True, False):
+        record(f"qkv_rotate_store, {'values that are the keys' if shared else 'values of their own (Katopel path)'}, {T} tokens, {nh} heads over {nkv} of {d}",
+               kernel_time(lambda: ops.qkv_rotate_store(wide, 0, bias, freq, 64, pos, pos, req0, q, pools[0], pools[1], nh, nkv, d, d, d,
+                                                        layout="half", values_are_keys=shared)),
+               T * ((nh + (1 if shared else 2) * nkv) * 4 + (nh + 2 * nkv) * 2) * d, "qkv_rotate_store" if shared else None)
+    del wide, pools, q
+    # ---- the dense feed-forward's up product with its activation, beside the gated product ----
+    ff = 8192
+    w, w_gated = rnd(ff, H, dtype=bf16), rnd(ff, H, dtype=bf16)
+    for m in (8192, 2048, 1024, 512, 256, 128, 64, 32, 16, 8, 1):
+        h = rnd(m, H, dtype=bf16)
+        flops, nbytes = 2 * m * ff * H, ff * H * 2 + m * (H + ff) * 2
+        record(f"up product with the square of relu, {m} x {H} -> {ff}",
+               kernel_time(lambda: gemm_bf16.linear_bf16_activated(h, w, None, "relu_squared")), nbytes, "gated_linear", flops=flops)
+        if m >= 64:
+            record(f"up product by the library, activation behind it, {m} x {H} -> {ff}",
+                   kernel_time(lambda: ops.activate(torch.mm(h, w.t()), "relu_squared")), nbytes, None, flops=flops)
+        act = torch.empty(m, ff // 2, dtype=bf16, device=dev)
+        record(f"gated_linear (Qwen2 path), {m} x {H} -> {ff}", kernel_time(lambda: ops.gated_linear(h, w_gated, act)), nbytes, None, flops=flops)
+    z = rnd(T, ff, dtype=bf16)
+    record(f"activate, {T} x {ff}", kernel_time(lambda: ops.activate(z, "relu_squared")), T * ff * 4, "silu_gate")
+    z2, half = rnd(T, 2 * ff, dtype=bf16), torch.empty(T, ff, dtype=bf16, device=dev)
+    record(f"silu_gate (Qwen2 path), {T} x {ff}", kernel_time(lambda: ops.silu_gate(z2, half)), T * ff * 6, None)
+    ops.raise_if_error()
+    print(json.dumps({
+        "metric": "prefill and decode tok/s of the Kerudra design beside Pufuzen at equal width, depth and parameters",
+        "unit": "tokens/s", "n_gpus": 1, "steps": steps, "warmup": args.warmup, "dtype": "bf16",
+        "data": "synthetic: random weights drawn on the device, uniform random token ids",
+        "config": {"sizes": KERUDRA_SIZES, "prefill_tokens": PREFILL_TOKENS, "decode_context": context,
                    "peaks": pk["source"], "hbm_gbs": pk["hbm_gbs"],
                    "l2": "kernels alone: inputs larger than L2 and a 256 MB write between timed launches"},
         "models": models, "kernels": kernels}))
