@@ -410,6 +410,67 @@ def test_segments_side_by_side_give_what_one_run_gives(heads, dim, vdim, segment
         m.check_state(slot, states)
 
 
+CHUNK_SIZES = [(3, 24, 16), (1, 6, 10), (2, 128, 128), (4, 64, 96), (2, 100, 8), (3, 7, 5), (1, 1, 1), (2, 32, 33), (1, 120, 63), (2, 32, 48)]
+
+
+@pytest.mark.parametrize("heads,dim,vdim", CHUNK_SIZES)
+def test_chunks_on_tensor_cores_carry_the_same_state(heads, dim, vdim):
+    """Portions cut in the middle of a chunk, on its border, of one token and of many chunks, three requests side by side
+    and an idle one: q, k and v as bfloat16 numbers, everything else to 32-bit accuracy (the state tells, the outputs
+    are rounded)."""
+    o, eps = ops(), 1e-4
+    lengths, slots = [200, 64, 331], [2, 0, 3]
+    cuts = [[0, 1, 64, 128, 131, 200], [0, 64], [0, 129, 193, 194, 330, 331]]
+    total = sum(lengths)
+    m = Memory(heads, dim, vdim, total, 110)
+    for name, lanes in (("q", dim), ("k", dim), ("v", vdim)):
+        part = m.proj[:, m.at[name]:m.at[name] + heads * lanes]
+        part.copy_(part.bfloat16().float())
+    m.state[1] = 7.0
+    out = torch.full((total, heads * vdim), float("nan"), dtype=torch.bfloat16, device=DEV)
+    starts = np.concatenate(([0], np.cumsum(lengths)))
+    assert o.mlstm_chunks_supported(dim, vdim)
+    for i in range(5):
+        rows, spans, who = [], [0], []
+        for r in range(3):
+            if i + 1 < len(cuts[r]):
+                rows += list(range(starts[r] + cuts[r][i], starts[r] + cuts[r][i + 1]))
+                spans.append(len(rows))
+                who.append(slots[r])
+        idx = torch.tensor(rows, device=DEV)
+        sub, spans, who = m.proj[idx].contiguous(), ints(spans + [spans[-1]]), ints(who + [0])
+        gates = torch.full((3, heads, len(rows) + 1), float("nan"), device=DEV)
+        start = torch.full((who.shape[0], heads), float("nan"), device=DEV)
+        o.mlstm_gates(sub, m.at["i"], m.at["f"], m.ib, m.fb, m.cap, heads, m.state, m.m_off, spans, who, gates, start)
+        y = torch.full((len(rows), heads * vdim), float("nan"), dtype=torch.bfloat16, device=DEV)
+        o.mlstm_chunks(sub, m.at["q"], m.at["k"], m.at["v"], m.at["g"], heads, dim, vdim, gates, start, m.gain, eps, m.state, spans, who, y)
+        out[idx] = y
+    for r in range(3):
+        want, states = m.plain(m.proj[starts[r]:starts[r + 1]], eps)
+        close(out[starts[r]:starts[r + 1]], want, torch.bfloat16, f"request {r}", 6e-3)
+        m.check_state(slots[r], states, 1e-5)
+    assert torch.all(m.state[1] == 7.0) and torch.all(m.state[4] == 0.0)
+
+
+@pytest.mark.parametrize("forget", [-14.0, -3.0, 14.0])
+def test_chunks_keep_their_digits_under_closed_and_open_gates(forget):
+    """Forget gates that all but close (their logarithms add up to hundreds inside a chunk and cancel) or stay open, for
+    every token: the state to 32-bit accuracy, and a write of the chunk before last that an open gate keeps."""
+    o, heads, dim, vdim, total, eps = ops(), 2, 64, 32, 300, 1e-4
+    m = Memory(heads, dim, vdim, total, 120, cap=15.0)
+    m.proj = m.proj.bfloat16().float()
+    m.fb.fill_(4.0 * forget)
+    gates, start = torch.empty(3, heads, total, device=DEV), torch.empty(1, heads, device=DEV)
+    spans, who = ints([0, total]), ints([1])
+    o.mlstm_gates(m.proj, m.at["i"], m.at["f"], m.ib, m.fb, m.cap, heads, m.state, m.m_off, spans, who, gates, start)
+    y = torch.empty(total, heads * vdim, dtype=torch.bfloat16, device=DEV)
+    o.mlstm_chunks(m.proj, m.at["q"], m.at["k"], m.at["v"], m.at["g"], heads, dim, vdim, gates, start, m.gain, eps, m.state, spans, who, y)
+    want, states = m.plain(m.proj, eps)
+    assert float(start.abs().max()) == 0.0
+    close(y, want, torch.bfloat16, "outputs", 6e-3)
+    m.check_state(1, states, 1e-5)
+
+
 def test_a_write_behind_a_thousand_tokens_and_a_maximum_that_starts_at_zero():
     """One token writes with an open input gate; every later one keeps (forget gate near one) and hardly writes; the last
     reads it back, through portions' borders.  And: with every input gate nearly shut the maximum falls from zero by the
@@ -465,7 +526,7 @@ def test_the_activation_as_a_kernel_of_its_own(activation, dtype):
 
 @pytest.mark.parametrize("activation", ["relu_squared", "gelu_pytorch_tanh"])
 @pytest.mark.parametrize("rows,n,k", [(1, 200, 96), (8, 72, 64), (16, 4096, 1024), (5, 8192, 2048), (20, 640, 512), (48, 256, 128), (48, 4104, 128),
-                                      (130, 384, 256), (256, 384, 256), (300, 1000, 264), (300, 37, 50), (9, 9, 14), (700, 2048, 512)])
+                                      (130, 384, 256), (256, 384, 256), (300, 1000, 264), (300, 37, 50), (9, 9, 14), (2300, 520, 136), (2048, 256, 64)])
 def test_the_activation_in_the_products_epilogue(rows, n, k, activation):
     """Whichever kernel the row count selects applies the activation to the 32-bit sums."""
     from tokenizer_b200.parts.linear import Linear
@@ -477,6 +538,27 @@ def test_the_activation_in_the_products_epilogue(rows, n, k, activation):
     close(Linear(w, bias).forward(a, activation=activation), want, torch.bfloat16, "with a bias", 1.5e-2)
     if rows < 50:
         close(Linear(w.float()).forward(a.float(), activation=activation), ACT[activation](double(a) @ double(w).t()), torch.float32, "float32")
+
+
+@pytest.mark.parametrize("rows,n,k", [(60, 256, 128), (300, 520, 264), (1000, 2048, 64)])
+def test_the_activation_in_the_tile_kernels_epilogue(rows, n, k):
+    """The tensor-core tile kernels of lone CTAs and of pairs, at sizes that other kernels usually take."""
+    o = ops()
+    a, w, bias = rnd(rows, k, seed=92, dtype=torch.bfloat16), rnd(n, k, seed=93, dtype=torch.bfloat16, scale=2.0 * k ** -0.5), rnd(n, seed=94)
+    z = double(a) @ double(w).t()
+    for b, add in ((None, 0.0), (bias, double(bias))):
+        for kind in (None, o.PAIR_PLAIN, o.PAIR_PLAIN_128):
+            out = torch.full((rows, n), float("nan"), dtype=torch.bfloat16, device=DEV)
+            if kind is None:
+                o.gemm_tcgen05(a, w, b, out, activation="relu_squared")
+            else:
+                o.gemm_tcgen05_pair(a, w, b, out, kind, "relu_squared")
+            close(out, ACT["relu_squared"](z + add), torch.bfloat16, str(kind), 1.5e-2)
+    plain_out = torch.empty(rows, n, dtype=torch.bfloat16, device=DEV)
+    o.gemm_tcgen05(a, w, None, plain_out)
+    close(plain_out, z, torch.bfloat16, "no activation", 1.5e-2)
+    with pytest.raises(ValueError):
+        o.gemm_tcgen05(a, w, None, torch.empty(rows, n, device=DEV), activation="relu_squared")       # a 32-bit result has no such epilogue
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])

@@ -169,9 +169,11 @@ TOKB200_API int tokb200_rotate_interleaved(void* x, int dtype, int heads, int he
 // latent_rotate_store: one projection's output row holds the key/value latent with its positional key part (c_at ..)
 // and, for every head, a query in the cache row's own lanes (q_at .., `row` a head: kv_rank lanes without position,
 // rot_dim with, the rest zero).  The latent is RMS-normed with its gain, the positional parts of the key and of every
-// query are rotated (lane 2i with lane 2i + 1), the key row goes to the cache, the queries to q_out.  A block a token,
-// a warp a row; the angles are formed in 64-bit and brought into one turn before sine and cosine, once a token.
-template <typename TO>
+// query are rotated (lane 2i with lane 2i + 1), the key row goes to the cache, the queries to q_out.  A block a token;
+// the angles are formed in 64-bit and brought into one turn before sine and cosine, once a token.  The key row is one
+// warp's; the queries are a warp's each, or, where everything comes in whole 4s on 16 bytes (QUADS), four lanes a
+// thread wherever they lie, asked for before the angles are waited for.
+template <typename TO, bool QUADS>
 __global__ void __launch_bounds__(256)
 latent_rotate_store_kernel(const float* __restrict__ proj, int ld, int c_at, int q_at, int heads, int kv_rank, int rot_dim,
                            int rot_dims, int row, const float* __restrict__ c_gain, float eps,
@@ -194,8 +196,40 @@ latent_rotate_store_kernel(const float* __restrict__ proj, int ld, int c_at, int
   pdl_wait();
   pdl_launch();
   if (r < 0) return;
-  __syncthreads();
   const float* in = proj + (size_t)t * ld;
+  if (QUADS) {
+    constexpr int DEEP = 4;
+    const int n = heads * row;
+    for (int base = threadIdx.x * 4; base < n; base += blockDim.x * 4 * DEEP) {
+      float4 v[DEEP];
+#pragma unroll
+      for (int d = 0; d < DEEP; ++d) {
+        const int i = base + d * blockDim.x * 4;
+        if (i < n) v[d] = *reinterpret_cast<const float4*>(in + q_at + i);
+      }
+      if (base == threadIdx.x * 4) __syncthreads();      // the angles (every thread comes by once: n is at least a thread's 4 lanes)
+#pragma unroll
+      for (int d = 0; d < DEEP; ++d) {
+        const int i = base + d * blockDim.x * 4;
+        if (i >= n) continue;
+        const int l = i % row - kv_rank;                 // inside the rotated part: 0 .. rot_dims - 1
+        if (l >= 0 && l < rot_dims) {
+          const float c0 = angles[l >> 1], s0 = angles[half + (l >> 1)], c1 = angles[(l >> 1) + 1], s1 = angles[half + (l >> 1) + 1];
+          v[d] = make_float4(v[d].x * c0 - v[d].y * s0, v[d].y * c0 + v[d].x * s0, v[d].z * c1 - v[d].w * s1,
+                             v[d].w * c1 + v[d].z * s1);
+        }
+        TO* dst = q_out + (size_t)t * n + i;
+        if (sizeof(TO) == 4) {
+          *reinterpret_cast<float4*>(dst) = v[d];
+        } else {
+          __nv_bfloat162 h[2] = {__floats2bfloat162_rn(v[d].x, v[d].y), __floats2bfloat162_rn(v[d].z, v[d].w)};
+          *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(h);
+        }
+      }
+    }
+  } else {
+    __syncthreads();
+  }
   // lane l of a rotated part that starts at `part`
   auto rotated = [&](const float* part, int l) {
     const float own = part[l];
@@ -203,7 +237,7 @@ latent_rotate_store_kernel(const float* __restrict__ proj, int ld, int c_at, int
     const float other = part[l ^ 1], c = angles[l >> 1], s = angles[half + (l >> 1)];
     return (l & 1) ? own * c + other * s : own * c - other * s;
   };
-  for (int item = warp; item <= heads; item += warps) {
+  for (int item = QUADS ? (warp == warps - 1 ? 0 : 1) : warp; item <= (QUADS ? 0 : heads); item += warps) {
     if (item == 0) {                          // the latent and the shared key part
       if (where < 0) continue;
       const float* c = in + c_at;
@@ -235,14 +269,22 @@ TOKB200_API int tokb200_latent_rotate_store(const float* proj, int ld, int c_at,
       row < kv_rank + rot_dim || c_at + kv_rank + rot_dim > ld || q_at + heads * row > ld || rot_dims > 8192 ||
       (rot_dims > 0 && inv_freq == nullptr))
     return TOKB200_BAD_SIZE;
-  const int warps = heads + 1 < 8 ? heads + 1 : 8;
+  const bool quads = heads * row >= 128 && ((row | kv_rank | rot_dims | q_at | ld) & 3) == 0 && (((uintptr_t)proj | (uintptr_t)q_out) & 15) == 0;
+  // QUADS: no more threads than there are quads of query lanes
+  const int warps = quads ? (heads * row / 128 < 8 ? heads * row / 128 : 8) : heads + 1 < 8 ? heads + 1 : 8;
   const size_t smem = (size_t)rot_dims * sizeof(float);
-#define LAUNCH(TO)                                                                                                     \
-  return launch_dependent(latent_rotate_store_kernel<TO>, dim3(n_rows), dim3(warps * 32), smem, stream, proj, ld, c_at, \
+#define LAUNCH(TO, QUADS)                                                                                              \
+  return launch_dependent(latent_rotate_store_kernel<TO, QUADS>, dim3(n_rows), dim3(warps * 32), smem, stream, proj, ld, c_at, \
                           q_at, heads, kv_rank, rot_dim, rot_dims, row, c_gain, eps, inv_freq, pos, row_req, slot,      \
                           (TO*)q_out, (TO*)pool)
-  if (out_dtype == TOKB200_F32) LAUNCH(float);
-  if (out_dtype == TOKB200_BF16) LAUNCH(__nv_bfloat16);
+  if (out_dtype == TOKB200_F32) {
+    if (quads) LAUNCH(float, true);
+    LAUNCH(float, false);
+  }
+  if (out_dtype == TOKB200_BF16) {
+    if (quads) LAUNCH(__nv_bfloat16, true);
+    LAUNCH(__nv_bfloat16, false);
+  }
 #undef LAUNCH
   return TOKB200_BAD_DTYPE;
 }
@@ -252,8 +294,9 @@ TOKB200_API int tokb200_latent_rotate_store(const float* proj, int ld, int c_at,
 // mixed [T, heads, row], w per head.  In bfloat16 (w [heads, vdim, row], row in whole 16s) a product on tensor cores
 // whose epilogue applies the gate: it is bound by reading mixed and gate, not by its arithmetic (row and vdim are a
 // hundred or so).  A tile is 64 lanes of a head by 64 rows (a warp 16 rows), or, with few rows, by 16 (a warp 16 lanes);
-// k goes through shared memory in pieces of 64.
-#define LV_K 64
+// k goes through shared memory in pieces of 128, every load of a piece in flight at once, and the gate is asked for with
+// the first piece.
+#define LV_K 128
 #define LV_PITCH (LV_K + 8)
 template <bool FEW>
 __global__ void __launch_bounds__(128)
@@ -267,17 +310,42 @@ latent_values_mma_kernel(const __nv_bfloat16* __restrict__ mixed, const __nv_bfl
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int row_in = FEW ? 0 : warp * 16, lane_in = FEW ? warp * 16 : 0;
   const __nv_bfloat16* wh = w + (size_t)head * vdim * row;
+  auto copy16 = [](__nv_bfloat16* dst, const __nv_bfloat16* src, bool ok) {      // zeros where there is nothing
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src),
+                 "r"(ok ? 16 : 0) : "memory");
+  };
   auto stage_w = [&](int k0) {
     for (int i = threadIdx.x; i < 64 * (LV_K / 8); i += 128) {
       const int l = i / (LV_K / 8), k = (i % (LV_K / 8)) * 8;
-      uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (l0 + l < vdim && k0 + k < row) v = *reinterpret_cast<const uint4*>(wh + (size_t)(l0 + l) * row + k0 + k);
-      *reinterpret_cast<uint4*>(&w_s[l][k]) = v;
+      const bool ok = l0 + l < vdim && k0 + k < row;
+      copy16(&w_s[l][k], ok ? wh + (size_t)(l0 + l) * row + k0 + k : wh, ok);
+    }
+  };
+  auto stage_a = [&](int k0) {
+    for (int i = threadIdx.x; i < ROWS * (LV_K / 8); i += 128) {
+      const int m = i / (LV_K / 8), k = (i % (LV_K / 8)) * 8;
+      const bool ok = t0 + m < n_rows && k0 + k < row;
+      copy16(&a_s[m][k], ok ? mixed + ((size_t)(t0 + m) * heads + head) * row + k0 + k : mixed, ok);
     }
   };
   stage_w(0);                                 // weights are written by no kernel of the step
   pdl_wait();
   pdl_launch();
+  stage_a(0);
+  const int g = lane >> 2, q = lane & 3;
+  const bool pairs = (vdim & 1) == 0 && (g_at & 1) == 0 && (ld & 1) == 0;
+  float2 z[TILES][2];                         // the gate's numbers for this thread's results
+#pragma unroll
+  for (int j = 0; j < TILES; ++j)
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int t = t0 + row_in + g + 8 * h, l = l0 + lane_in + 8 * j + 2 * q;
+      z[j][h] = make_float2(0.f, 0.f);
+      if (t >= n_rows || l >= vdim) continue;
+      const float* from = gate + (size_t)t * ld + g_at + head * vdim + l;
+      if (pairs) z[j][h] = *reinterpret_cast<const float2*>(from);
+      else z[j][h] = make_float2(from[0], l + 1 < vdim ? from[1] : 0.f);
+    }
   float acc[TILES][4];
 #pragma unroll
   for (int j = 0; j < TILES; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
@@ -285,17 +353,14 @@ latent_values_mma_kernel(const __nv_bfloat16* __restrict__ mixed, const __nv_bfl
     if (k0) {
       __syncthreads();                        // the piece before has been read
       stage_w(k0);
+      stage_a(k0);
     }
-    for (int i = threadIdx.x; i < ROWS * (LV_K / 8); i += 128) {
-      const int m = i / (LV_K / 8), k = (i % (LV_K / 8)) * 8;
-      uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (t0 + m < n_rows && k0 + k < row)
-        v = *reinterpret_cast<const uint4*>(mixed + ((size_t)(t0 + m) * heads + head) * row + k0 + k);
-      *reinterpret_cast<uint4*>(&a_s[m][k]) = v;
-    }
+    asm volatile("cp.async.wait_all;" ::: "memory");
     __syncthreads();
+    const int k_end = row - k0 < LV_K ? row - k0 : LV_K;      // rows come in whole 16s
 #pragma unroll
     for (int k = 0; k < LV_K; k += 16) {
+      if (k >= k_end) break;
       unsigned a[4];
       const unsigned from = (unsigned)__cvta_generic_to_shared(&a_s[row_in + (lane & 15)][k + (lane >> 4) * 8]);
       asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
@@ -315,21 +380,19 @@ latent_values_mma_kernel(const __nv_bfloat16* __restrict__ mixed, const __nv_bfl
       }
     }
   }
-  const int g = lane >> 2, q = lane & 3;
 #pragma unroll
   for (int j = 0; j < TILES; ++j)
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       const int t = t0 + row_in + g + 8 * h, l = l0 + lane_in + 8 * j + 2 * q;
       if (t >= n_rows || l >= vdim) continue;
-      const float* z = gate + (size_t)t * ld + g_at + head * vdim + l;
       __nv_bfloat16* o = out + ((size_t)t * heads + head) * vdim + l;
-      const float v0 = acc[j][2 * h] / (1.0f + expf(-z[0]));
+      const float v0 = acc[j][2 * h] / (1.0f + expf(-z[j][h].x)), v1 = acc[j][2 * h + 1] / (1.0f + expf(-z[j][h].y));
       if ((vdim & 1) == 0) {
-        *reinterpret_cast<__nv_bfloat162*>(o) = __floats2bfloat162_rn(v0, acc[j][2 * h + 1] / (1.0f + expf(-z[1])));
+        *reinterpret_cast<__nv_bfloat162*>(o) = __floats2bfloat162_rn(v0, v1);
       } else {
         o[0] = __float2bfloat16_rn(v0);
-        if (l + 1 < vdim) o[1] = __float2bfloat16_rn(acc[j][2 * h + 1] / (1.0f + expf(-z[1])));
+        if (l + 1 < vdim) o[1] = __float2bfloat16_rn(v1);
       }
     }
 }
@@ -364,7 +427,7 @@ TOKB200_API int tokb200_latent_values(const void* mixed, const void* w, const fl
                             (size_t)row * sizeof(float), stream, (const float*)mixed, (const float*)w, gate, ld, g_at, heads,
                             vdim, row, (float*)out);
   if (dtype != TOKB200_BF16) return TOKB200_BAD_DTYPE;
-  if (row % 16 || (((uintptr_t)mixed | (uintptr_t)w) & 15) || ((uintptr_t)out & 3)) return TOKB200_BAD_ALIGNMENT;
+  if (row % 16 || (((uintptr_t)mixed | (uintptr_t)w) & 15) || ((uintptr_t)out & 3) || ((uintptr_t)gate & 7)) return TOKB200_BAD_ALIGNMENT;
   const bool few = n_rows <= 64;
   const dim3 grid((n_rows + (few ? 15 : 63)) / (few ? 16 : 64), heads, (vdim + 63) / 64);
 #define LAUNCH(FEW)                                                                                              \

@@ -13,8 +13,9 @@
 //                   exp(-m), one of each a token and head; the rest of the recurrence is then linear in (S, n)
 //   mlstm_scan      that recurrence on the scan that matrix recurrences share (matrix_scan.cuh): n is the column
 //                   of ones, its product with q comes back as one number a token and head
-//   mlstm_out_norm  the division, the norm, the gain and the gate: a warp a (token, head)
+//   mlstm_out_norm  the division, the norm, the gain and the gate: a warp a (token, head), or a few of them
 //   mlstm_step      all of it for a step of single tokens, a block a (row, head)
+// (In bfloat16 long portions take the scan and the norm in chunks on tensor cores instead: mlstm_chunks.cu.)
 //
 // A slot: [heads, vdim + 1, dim] (S transposed, n behind the last column), then m [heads].
 #include "matrix_scan.cuh"
@@ -33,12 +34,15 @@ __device__ __forceinline__ MlStep ml_then(MlStep first, MlStep second) {
   return {first.a + second.a, fmaxf(first.b + second.a, second.b)};
 }
 
-// proj: [T, ld]; columns i_at .. + heads and f_at .. + heads are the gates' products.  A block a (head, request).
+// proj: [T, ld]; columns i_at .. + heads and f_at .. + heads are the gates' products.  A block a (head, request).  With
+// `start` (float32 [requests, heads]) the three numbers a token and head are f, i and m themselves instead, and `start`
+// receives the m in front of the step's rows: what the form in chunks works from.
 __global__ void mlstm_gates_kernel(const float* __restrict__ proj, int ld, int i_at, int f_at,
                                    const float* __restrict__ i_bias, const float* __restrict__ f_bias, float cap,
                                    float* __restrict__ state, long long stride, int m_off, const int* __restrict__ q_start,
                                    const int* __restrict__ state_slot, float* __restrict__ keep,
-                                   float* __restrict__ add, float* __restrict__ floor_out, long long gate_ld) {
+                                   float* __restrict__ add, float* __restrict__ floor_out, long long gate_ld,
+                                   float* __restrict__ start_out) {
   __shared__ float warp_a[32], warp_b[32];
   __shared__ float tops[1024];
   const int head = blockIdx.x, r = blockIdx.y;
@@ -50,6 +54,7 @@ __global__ void mlstm_gates_kernel(const float* __restrict__ proj, int ld, int i
   if (n <= 0) return;
   float* m_state = state + (size_t)state_slot[r] * stride + m_off + head;
   float carry = *m_state;
+  if (start_out && threadIdx.x == 0) start_out[(size_t)r * gridDim.x + head] = carry;
   for (int base = 0; base < n; base += blockDim.x) {
     const int at = base + threadIdx.x;
     const bool live = at < n;
@@ -80,9 +85,9 @@ __global__ void mlstm_gates_kernel(const float* __restrict__ proj, int ld, int i
       // the neighbour's own number: what one token's S is divided by is what the next token's keep starts from
       const float before = threadIdx.x == 0 ? carry : tops[threadIdx.x - 1];
       const size_t o = (size_t)head * gate_ld + first + at;
-      keep[o] = expf(lf + before - top);
-      add[o] = expf(li - top);
-      floor_out[o] = expf(-top);
+      keep[o] = start_out ? lf : expf(lf + before - top);
+      add[o] = start_out ? li : expf(li - top);
+      floor_out[o] = start_out ? top : expf(-top);
     }
     carry = tops[warps * 32 - 1];                         // idle threads behind the last token carry its m on
     __syncthreads();                                      // tops and the warps' sums are written again by the next run
@@ -93,14 +98,15 @@ __global__ void mlstm_gates_kernel(const float* __restrict__ proj, int ld, int i
 TOKB200_API int tokb200_mlstm_gates(const float* proj, int ld, int i_at, int f_at, const float* i_bias,
                                     const float* f_bias, float cap, int heads, float* state, long long stride, int m_off,
                                     const int* q_start, const int* state_slot, int n_requests, int n_rows, float* keep,
-                                    float* add, float* floor_out, long long gate_ld, cudaStream_t stream) {
+                                    float* add, float* floor_out, long long gate_ld, float* start, cudaStream_t stream) {
   if (n_requests <= 0 || n_rows <= 0) return TOKB200_OK;
   if (heads <= 0 || n_requests > 65535 || cap <= 0.f || i_at + heads > ld || f_at + heads > ld || gate_ld < n_rows ||
       m_off + heads > stride)
     return TOKB200_BAD_SIZE;
   const int threads = n_rows >= 1024 ? 1024 : n_rows >= 256 ? 256 : 64;
   return launch_dependent(mlstm_gates_kernel, dim3(heads, n_requests), dim3(threads), 0, stream, proj, ld, i_at, f_at,
-                          i_bias, f_bias, cap, state, stride, m_off, q_start, state_slot, keep, add, floor_out, gate_ld);
+                          i_bias, f_bias, cap, state, stride, m_off, q_start, state_slot, keep, add, floor_out, gate_ld,
+                          start);
 }
 
 // proj: float32 [T, ld]: q (heads * dim), k (heads * dim) and v (heads * vdim) at their columns.  y [T, heads, vdim]
@@ -122,65 +128,85 @@ TOKB200_API int tokb200_mlstm_scan(const float* proj, int ld, int q_at, int k_at
 }
 
 // y [T, heads, vdim], yn [T, heads], floors [heads, gate_ld]; the gate's products at columns g_at .. of proj.
+// SPAN > 0: heads of up to 128 SPAN lanes in whole 4s with everything on 16 bytes: a warp takes 4 / SPAN of them, every
+// load asked for before the first is used.
 #define ML_NORM_WARPS 8
-template <typename TO, bool QUADS>
+template <typename TO, int SPAN>
 __global__ void __launch_bounds__(ML_NORM_WARPS * 32)
 mlstm_out_norm_kernel(const float* __restrict__ y, const float* __restrict__ yn, const float* __restrict__ floors,
                       long long gate_ld, const float* __restrict__ proj, int ld, int g_at,
                       const float* __restrict__ gain, float eps, int heads, int vdim, const int* __restrict__ row_req,
                       TO* __restrict__ out, int n_rows) {
+  constexpr int ITEMS = SPAN ? 4 / SPAN : 1;
   const int lane = threadIdx.x & 31;
-  const int item = blockIdx.x * ML_NORM_WARPS + (threadIdx.x >> 5);
-  const int t = item / heads, head = item % heads;
+  const int first = (blockIdx.x * ML_NORM_WARPS + (threadIdx.x >> 5)) * ITEMS;
   pdl_wait();
   pdl_launch();
-  if (t >= n_rows || row_req[t] < 0) return;
-  const float* yr = y + ((size_t)t * heads + head) * vdim;
-  const float* gr = proj + (size_t)t * ld + g_at + head * vdim;
-  const float* wr = gain + head * vdim;
-  TO* o = out + ((size_t)t * heads + head) * vdim;
-  const float inv_den = 1.0f / (fmaxf(fabsf(yn[(size_t)t * heads + head]), floors[(size_t)head * gate_ld + t]) + ML_EPS);
-  float squares = 0.f;
-  if (QUADS) {                                            // up to 512 lanes in whole 4s, everything on 16 bytes
-    float4 kept[4], gate[4];
+  if (SPAN) {
+    constexpr int WIDE = SPAN ? SPAN : 1;
+    float4 kept[ITEMS][WIDE], gate[ITEMS][WIDE];
+    float den[ITEMS];
+    int token[ITEMS];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int l = (lane + 32 * j) * 4;
-      kept[j] = gate[j] = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (l < vdim) {
-        kept[j] = *reinterpret_cast<const float4*>(yr + l);
-        gate[j] = *reinterpret_cast<const float4*>(gr + l);
+    for (int k = 0; k < ITEMS; ++k) {
+      const int t = (first + k) / heads, head = first + k - t * heads;
+      const bool on = t < n_rows && row_req[t] >= 0;
+      token[k] = on ? t : -1;
+      den[k] = on ? fmaxf(fabsf(yn[(size_t)t * heads + head]), floors[(size_t)head * gate_ld + t]) : 1.f;
+#pragma unroll
+      for (int j = 0; j < WIDE; ++j) {
+        const int l = (lane + 32 * j) * 4;
+        kept[k][j] = gate[k][j] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (on && l < vdim) {
+          kept[k][j] = *reinterpret_cast<const float4*>(y + ((size_t)t * heads + head) * vdim + l);
+          gate[k][j] = *reinterpret_cast<const float4*>(proj + (size_t)t * ld + g_at + head * vdim + l);
+        }
       }
     }
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      kept[j].x *= inv_den; kept[j].y *= inv_den; kept[j].z *= inv_den; kept[j].w *= inv_den;
-      squares += fmaf(kept[j].x, kept[j].x, fmaf(kept[j].y, kept[j].y, fmaf(kept[j].z, kept[j].z, kept[j].w * kept[j].w)));
-    }
-    const float inv = 1.0f / sqrtf(warp_sum(squares) / (float)vdim + eps);
+    for (int k = 0; k < ITEMS; ++k) {
+      if (token[k] < 0) continue;             // the same for the whole warp
+      const int head = first + k - token[k] * heads;
+      const float inv_den = 1.0f / (den[k] + ML_EPS);
+      float squares = 0.f;
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int l = (lane + 32 * j) * 4;
-      if (l < vdim) {
-        const float4 w = *reinterpret_cast<const float4*>(wr + l);
-        const float v[4] = {kept[j].x * inv * w.x * ml_sigmoid(gate[j].x), kept[j].y * inv * w.y * ml_sigmoid(gate[j].y),
-                            kept[j].z * inv * w.z * ml_sigmoid(gate[j].z), kept[j].w * inv * w.w * ml_sigmoid(gate[j].w)};
+      for (int j = 0; j < WIDE; ++j) {
+        float4& v = kept[k][j];
+        v.x *= inv_den; v.y *= inv_den; v.z *= inv_den; v.w *= inv_den;
+        squares += fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
+      }
+      const float inv = 1.0f / sqrtf(warp_sum(squares) / (float)vdim + eps);
+#pragma unroll
+      for (int j = 0; j < WIDE; ++j) {
+        const int l = (lane + 32 * j) * 4;
+        if (l >= vdim) continue;
+        const float4 w = *reinterpret_cast<const float4*>(gain + head * vdim + l), v = kept[k][j], g = gate[k][j];
+        const float r[4] = {v.x * inv * w.x * ml_sigmoid(g.x), v.y * inv * w.y * ml_sigmoid(g.y),
+                            v.z * inv * w.z * ml_sigmoid(g.z), v.w * inv * w.w * ml_sigmoid(g.w)};
+        TO* o = out + ((size_t)token[k] * heads + head) * vdim + l;
         if (sizeof(TO) == 4) {
-          *reinterpret_cast<float4*>(o + l) = make_float4(v[0], v[1], v[2], v[3]);
+          *reinterpret_cast<float4*>(o) = make_float4(r[0], r[1], r[2], r[3]);
         } else {
-          __nv_bfloat162 h[2] = {__floats2bfloat162_rn(v[0], v[1]), __floats2bfloat162_rn(v[2], v[3])};
-          *reinterpret_cast<uint2*>(o + l) = *reinterpret_cast<const uint2*>(h);
+          __nv_bfloat162 h[2] = {__floats2bfloat162_rn(r[0], r[1]), __floats2bfloat162_rn(r[2], r[3])};
+          *reinterpret_cast<uint2*>(o) = *reinterpret_cast<const uint2*>(h);
         }
       }
     }
     return;
   }
+  const int t = first / heads, head = first % heads;
+  if (t >= n_rows || row_req[t] < 0) return;
+  const float* yr = y + ((size_t)t * heads + head) * vdim;
+  const float* gr = proj + (size_t)t * ld + g_at + head * vdim;
+  TO* o = out + ((size_t)t * heads + head) * vdim;
+  const float inv_den = 1.0f / (fmaxf(fabsf(yn[(size_t)t * heads + head]), floors[(size_t)head * gate_ld + t]) + ML_EPS);
+  float squares = 0.f;
   for (int l = lane; l < vdim; l += 32) {
     const float v = yr[l] * inv_den;
     squares = fmaf(v, v, squares);
   }
   const float inv = 1.0f / sqrtf(warp_sum(squares) / (float)vdim + eps);
-  for (int l = lane; l < vdim; l += 32) o[l] = from_float<TO>(yr[l] * inv_den * inv * wr[l] * ml_sigmoid(gr[l]));
+  for (int l = lane; l < vdim; l += 32) o[l] = from_float<TO>(yr[l] * inv_den * inv * gain[head * vdim + l] * ml_sigmoid(gr[l]));
 }
 
 TOKB200_API int tokb200_mlstm_out_norm(const float* y, const float* yn, const float* floors, long long gate_ld,
@@ -189,21 +215,22 @@ TOKB200_API int tokb200_mlstm_out_norm(const float* y, const float* yn, const fl
                                        cudaStream_t stream) {
   if (n_rows <= 0) return TOKB200_OK;
   if (heads <= 0 || vdim <= 0 || g_at + heads * vdim > ld || gate_ld < n_rows) return TOKB200_BAD_SIZE;
-  const size_t items = (size_t)n_rows * heads;
-  const dim3 grid((unsigned)((items + ML_NORM_WARPS - 1) / ML_NORM_WARPS)), block(ML_NORM_WARPS * 32);
   const bool quads = vdim % 4 == 0 && vdim <= 512 && ld % 4 == 0 && g_at % 4 == 0 &&
                      (((uintptr_t)y | (uintptr_t)proj | (uintptr_t)gain | (uintptr_t)out) & 15) == 0;
-#define LAUNCH(TO, QUADS)                                                                                               \
-  return launch_dependent(mlstm_out_norm_kernel<TO, QUADS>, grid, block, 0, stream, y, yn, floors, gate_ld, proj, ld, g_at, \
+  const int span = !quads ? 0 : vdim <= 128 ? 1 : vdim <= 256 ? 2 : 4;
+  const size_t items = (size_t)n_rows * heads, a_block = (size_t)ML_NORM_WARPS * (span ? 4 / span : 1);
+  const dim3 grid((unsigned)((items + a_block - 1) / a_block)), block(ML_NORM_WARPS * 32);
+#define LAUNCH(TO, SPAN)                                                                                               \
+  return launch_dependent(mlstm_out_norm_kernel<TO, SPAN>, grid, block, 0, stream, y, yn, floors, gate_ld, proj, ld, g_at, \
                           gain, eps, heads, vdim, row_req, (TO*)out, n_rows)
-  if (out_dtype == TOKB200_F32) {
-    if (quads) LAUNCH(float, true);
-    LAUNCH(float, false);
-  }
-  if (out_dtype == TOKB200_BF16) {
-    if (quads) LAUNCH(__nv_bfloat16, true);
-    LAUNCH(__nv_bfloat16, false);
-  }
+#define BY_SPAN(TO)             \
+  if (span == 0) LAUNCH(TO, 0); \
+  if (span == 1) LAUNCH(TO, 1); \
+  if (span == 2) LAUNCH(TO, 2); \
+  LAUNCH(TO, 4)
+  if (out_dtype == TOKB200_F32) { BY_SPAN(float); }
+  if (out_dtype == TOKB200_BF16) { BY_SPAN(__nv_bfloat16); }
+#undef BY_SPAN
 #undef LAUNCH
   return TOKB200_BAD_DTYPE;
 }

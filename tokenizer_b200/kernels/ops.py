@@ -1693,10 +1693,11 @@ MLSTM_MAX_DIM = 256
 
 
 def mlstm_gates(proj: torch.Tensor, i_at: int, f_at: int, i_bias, f_bias, cap: float, heads: int, state: torch.Tensor,
-                m_off: int, q_start, state_slot, gates: torch.Tensor) -> None:
+                m_off: int, q_start, state_slot, gates: torch.Tensor, start: Optional[torch.Tensor] = None) -> None:
     """The running maximum of every request's rows (`state` [slots, n]: it starts from and ends in the heads' numbers at
     m_off), and `gates` float32 [3, heads, >= T]: what a token's matrix is kept by, what its write is weighed by, and
-    exp(-maximum)."""
+    exp(-maximum).  With `start` (float32 [requests, heads], receives the maxima in front of the rows) `gates` holds the
+    logarithms of the forget and input gates and the maxima themselves, as `mlstm_chunks` wants them."""
     if proj.dtype != torch.float32 or gates.dtype != torch.float32 or gates.shape[:2] != (3, heads) or \
             state.dtype != torch.float32 or state.dim() != 2 or \
             any(v.dtype != torch.float32 or v.numel() != heads for v in (i_bias, f_bias)):
@@ -1704,7 +1705,34 @@ def mlstm_gates(proj: torch.Tensor, i_at: int, f_at: int, i_bias, f_bias, cap: f
     _check(_lib("mlstm").tokb200_mlstm_gates(
         _sliced_ptr(proj), _i(_ld(proj)), _i(i_at), _i(f_at), _ptr(i_bias), _ptr(f_bias), _f(cap), _i(heads), _ptr(state),
         _ll(state.shape[1]), _i(m_off), _ptr(q_start), _ptr(state_slot), _i(q_start.shape[0] - 1), _i(proj.shape[0]),
-        _ptr(gates[0]), _ptr(gates[1]), _ptr(gates[2]), _ll(gates.shape[2]), _stream()), "mlstm_gates")
+        _ptr(gates[0]), _ptr(gates[1]), _ptr(gates[2]), _ll(gates.shape[2]), _ptr(start), _stream()), "mlstm_gates")
+
+
+def mlstm_chunks_supported(dim: int, vdim: int) -> bool:
+    """Whether the form in chunks takes heads of these sizes."""
+    return bool(_lib("mlstm_chunks").tokb200_mlstm_chunks_supported(_i(dim), _i(vdim)))
+
+
+def mlstm_chunks(proj: torch.Tensor, q_at: int, k_at: int, v_at: int, g_at: int, heads: int, dim: int, vdim: int,
+                 gates: torch.Tensor, start: torch.Tensor, gain, eps: float, state: torch.Tensor, q_start, state_slot,
+                 out: torch.Tensor) -> None:
+    """What `mlstm_scan` and `mlstm_out_norm` do, in chunks of 64 tokens on tensor cores (csrc/mlstm_chunks.cu), q, k and v
+    as bfloat16 operands; `gates` and `start` from `mlstm_gates`.  `out` bfloat16 [T, heads * vdim]."""
+    n, n_requests = proj.shape[0], q_start.shape[0] - 1
+    if proj.dtype != torch.float32 or out.dtype != torch.bfloat16 or tuple(out.shape) != (n, heads * vdim) or \
+            gates.dtype != torch.float32 or gates.shape[:2] != (3, heads) or gates.shape[2] < n or gain.numel() != heads * vdim or \
+            start.dtype != torch.float32 or start.numel() != n_requests * heads or state.dtype != torch.float32 or \
+            state.dim() != 2 or heads * (vdim + 1) * dim > state.shape[1]:
+        raise ValueError("mlstm_chunks: sizes of the product, the gates, the state or the output disagree")
+    places = n // 64 + n_requests
+    sums = torch.empty(places * heads * (vdim + 1) * dim, dtype=torch.float32, device=proj.device)
+    decay = torch.empty(places * heads, dtype=torch.float32, device=proj.device)
+    _check(_lib("mlstm_chunks").tokb200_mlstm_chunks(
+        _sliced_ptr(proj), _i(_ld(proj)), _i(q_at), _i(k_at), _i(v_at), _i(g_at), _i(heads), _i(dim), _i(vdim), _f(dim ** -0.5),
+        _ptr(gates[0]), _ptr(gates[1]), _ptr(gates[2]), _ll(gates.shape[2]), _ptr(start), _ptr(q_start), _ptr(state_slot),
+        _i(n_requests), _i(n), _ptr(state), _ll(state.shape[1]), _ptr(sums), _ptr(decay), _ptr(gain), _f(eps), _ptr(out),
+        _stream()), "mlstm_chunks")
+    counter.launches += 2
 
 
 def mlstm_scan(proj: torch.Tensor, q_at: int, k_at: int, v_at: int, heads: int, dim: int, vdim: int, gates: torch.Tensor,

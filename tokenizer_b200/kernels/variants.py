@@ -29,6 +29,7 @@ def all_variants():
         ("short_conv.cu", (), ()),
         ("mamba2.cu", (), ()),
         ("mlstm.cu", (), ()),
+        ("mlstm_chunks.cu", (), ()),
         ("streams.cu", (), ()),
     ]
     for head_dim in (16, 32, 48, 64, 128):

@@ -186,10 +186,14 @@ def linear_bf16(a: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tens
     return out
 
 
+ACTIVATED_ROWS = 2048     # from here on the product with its activation goes to pairs of CTAs
+
+
 def linear_bf16_activated(a: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], activation: str) -> torch.Tensor:
-    """act(a[M,K] weight[N,K]^T (+ bias)) as bfloat16 [M,N]: the activation in the epilogue of whichever kernel of the
-    framework the row count selects, on the 32-bit sums; where the vendor library's product leads (65 to LIBRARY_ROWS - 1
-    rows) or no such kernel takes the sizes, a kernel of its own behind the product."""
+    """act(a[M,K] weight[N,K]^T (+ bias)) as bfloat16 [M,N].  Few and many rows: the activation in the epilogue of the
+    framework's own kernel, on the 32-bit sums.  In between the vendor library's product with the activation's own kernel
+    behind it leads (2,048 -> 8,192, us with / against the own kernel: 64 rows 33 / 39, 256 rows 33 / 43, 1,024 rows
+    48 / 54, 2,048 rows 76 / 76, 8,192 rows 222 / 199).  TOKB200_GEMM=own keeps every product on the own kernels."""
     M, K = a.shape
     N = weight.shape[0]
     out = torch.empty((M, N), dtype=torch.bfloat16, device=a.device)
@@ -200,11 +204,11 @@ def linear_bf16_activated(a: torch.Tensor, weight: torch.Tensor, bias: Optional[
     if ops.linear_small_m_supported(M, K) and (M <= ops.SMALL_M_ROWS or N < 4096):
         ops.linear_small_m(a, weight, bias, out, 1, activation)
         return out
-    if ops.gemm_tcgen05_supported(M, N, K) and N % 8 == 0 and os.environ.get("TOKB200_GEMM", "") != "library":
-        if ops._PAIR and M >= LIBRARY_ROWS:
+    choice = os.environ.get("TOKB200_GEMM", "")
+    if ops.gemm_tcgen05_supported(M, N, K) and N % 8 == 0 and choice != "library" and (M >= ACTIVATED_ROWS or choice == "own"):
+        if ops._PAIR and M >= 256:
             ops.gemm_tcgen05_pair(a, weight, bias, out, ops.PAIR_PLAIN, activation)
-            return out
-        if M <= 64 or M >= LIBRARY_ROWS or os.environ.get("TOKB200_GEMM", "") == "own":
+        else:
             ops.gemm_tcgen05(a, weight, bias, out, activation=activation)
-            return out
+        return out
     return ops.activate(linear_bf16(a, weight, bias, torch.bfloat16), activation)

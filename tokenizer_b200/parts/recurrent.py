@@ -415,6 +415,12 @@ class Mamba2:
         return self.out.forward(gated, partials_ok=True)
 
 
+# A step whose longest portion has this many tokens runs the matrix memory in chunks (bfloat16); TOKB200_MEMORY_CHUNKS=0
+# keeps every portion on the scan
+MEMORY_CHUNKS_FROM = 64
+_MEMORY_CHUNKS = os.environ.get("TOKB200_MEMORY_CHUNKS", "1") != "0"
+
+
 class MatrixMemory:
     """A matrix memory with exponential gates (the mLSTM).  From the mixer's input h: q = Wq h dim^(-1/2), k = Wk h (heads x
     dim), v = Wv h (heads x vdim); per head the logarithms of two gates, each squashed into (-cap, cap) by a tanh:
@@ -427,7 +433,8 @@ class MatrixMemory:
     `.b`), `.norm`, `.o`.
 
     The stacked input product is written in float32; everything behind it but the output projection's operand is 32-bit
-    (`csrc/mlstm.cu`).  Per request it keeps, in one state slot: the heads' matrices with n behind their columns
+    (`csrc/mlstm.cu`).  In bfloat16 long portions run in chunks on tensor cores (`csrc/mlstm_chunks.cu`): there q, k and v
+    are rounded to bfloat16 operands, and the state and every weight that meets them stays 32-bit.  Per request it keeps, in one state slot: the heads' matrices with n behind their columns
     ([heads, vdim + 1, dim]), then the running maxima."""
 
     graph_safe = True    # launches depend on device-side metadata alone
@@ -462,12 +469,17 @@ class MatrixMemory:
         self.out = Linear(runtime.matrix(store.get(x + ".o")))
         self.m_off = self.heads * (self.vdim + 1) * self.dim
         self.state_floats = -(-(self.m_off + self.heads) // 4) * 4
+        self.chunked = runtime.dtype == torch.bfloat16 and _MEMORY_CHUNKS and self.dim <= 128 and self.vdim <= 128
 
     def cache_need(self):
         return CacheNeed(state=StateNeed((self.state_floats,)))
 
+    def _in_chunks(self, longest):
+        return self.chunked and longest >= MEMORY_CHUNKS_FROM
+
     def shape_key(self, q_lens):
-        return "memory1" if max(q_lens) == 1 else "memory"      # the kernels' choice
+        longest = max(q_lens)
+        return "memory1" if longest == 1 else "memory_chunks" if self._in_chunks(longest) else "memory"     # the kernels' choice
 
     def streamed_weights(self):
         return [self.inputs.weight, self.out.weight]
@@ -483,8 +495,14 @@ class MatrixMemory:
                            ctx.state_slot, y)
             return self.out.forward(y, partials_ok=True)
         gates = torch.empty((3, heads, n), dtype=torch.float32, device=proj.device)
+        start = torch.empty((ctx.q_start.shape[0] - 1, heads), dtype=torch.float32, device=proj.device) \
+            if self._in_chunks(ctx.max_q_len) else None
         ops.mlstm_gates(proj, at["i"], at["f"], self.i_bias, self.f_bias, self.cap, heads, cache.state, self.m_off,
-                        ctx.q_start, ctx.state_slot, gates)
+                        ctx.q_start, ctx.state_slot, gates, start)
+        if start is not None:
+            ops.mlstm_chunks(proj, at["q"], at["k"], at["v"], at["g"], heads, self.dim, self.vdim, gates, start, self.gain,
+                             self.eps, cache.state, ctx.q_start, ctx.state_slot, y)
+            return self.out.forward(y, partials_ok=True)
         raw = torch.empty((n, heads * self.vdim), dtype=torch.float32, device=proj.device)
         norm = torch.empty((n, heads), dtype=torch.float32, device=proj.device)
         ops.mlstm_scan(proj, at["q"], at["k"], at["v"], heads, self.dim, self.vdim, gates, cache.state, ctx.q_start,
