@@ -1912,6 +1912,13 @@ def run_kerudra(args):
         record(f"mlstm_scan, {where}, {heads} heads of {dim} x {vdim}",
                kernel_time(lambda: ops.mlstm_scan(proj, at["q"], at["k"], at["v"], heads, dim, vdim, gates, state, spans, slots, y32, yn)),
                T * heads * (2 * dim + 2 * vdim) * 4, "mamba2_scan", flops=T * heads * dim * (vdim + 1) * 6)
+        start = torch.zeros(requests, heads, device=dev)
+        ops.mlstm_gates(proj, at["i"], at["i"] + heads, ib, fb, 15.0, heads, state, m_off, spans, slots, gates, start)
+        record(f"mlstm_chunks (scan and output norm), {where}, {heads} heads of {dim} x {vdim}",
+               kernel_time(lambda: ops.mlstm_chunks(proj, at["q"], at["k"], at["v"], at["g"], heads, dim, vdim, gates, start, gain, 1e-6,
+                                                    state, spans, slots, y16)),
+               T * heads * (2 * dim * 4 + 2 * vdim * 4 + vdim * 2), "mamba2_scan, mamba2_out_norm", flops=T * heads * dim * (vdim + 1) * 6)
+        ops.mlstm_gates(proj, at["i"], at["i"] + heads, ib, fb, 15.0, heads, state, m_off, spans, slots, gates)
         s_state = torch.zeros(requests, s_heads * s_vdim * n_state, device=dev)
         record(f"mamba2_scan (Vizonex path), {where}, {s_heads} heads of {n_state} x {s_vdim}",
                kernel_time(lambda: ops.mamba2_scan(xbc, s_proj, 0, zeros, zeros, ones, s_heads, groups, s_vdim, n_state, s_state, spans, slots, s_y)),

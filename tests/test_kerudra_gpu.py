@@ -715,6 +715,18 @@ def test_mixed_batches_on_pages_and_slots_that_are_used_again(model, dtype, live
     compare(got, want, dtype, "mixed")
 
 
+@pytest.mark.parametrize("longest", [2, 20])
+def test_mixed_batches_with_portions_in_chunks(model, longest, monkeypatch):
+    """Portions that usually run on the scan, down to two tokens, in chunks on tensor cores, single tokens of others
+    beside them."""
+    from tokenizer_b200.parts import recurrent
+    monkeypatch.setattr(recurrent, "MEMORY_CHUNKS_FROM", longest)
+    folder, cfg, page, requests, want = model
+    steps, peak = ru.steps_mixed(requests, max_live=3, seed=7)
+    got = ru.collect(steps, replay(folder, "bfloat16", steps, peak, page, max_requests=3))
+    compare(got, want, "bfloat16", "mixed, in chunks")
+
+
 def test_sizes_that_tiny_models_make_equal_or_one(tmp_path_factory):
     """One head, one lane of most things; models of one kind of mixer alone (no keys kept at all, no matrices kept at
     all); a loop over every layer; no feed-forward anywhere; eight streams."""

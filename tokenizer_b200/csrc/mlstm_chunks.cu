@@ -90,8 +90,14 @@ __device__ __forceinline__ void mc_gates(const McArgs& a, const McChunk& m, int 
   const int lane = threadIdx.x;
   const size_t at = (size_t)head * a.gate_ld + m.first;
   double f[2];
+  float top[2], in[2];
 #pragma unroll
-  for (int e = 0; e < 2; ++e) f[e] = 2 * lane + e < m.rows ? (double)a.log_f[at + 2 * lane + e] : 0.0;
+  for (int e = 0; e < 2; ++e) {
+    const bool on = 2 * lane + e < m.rows;
+    f[e] = on ? (double)a.log_f[at + 2 * lane + e] : 0.0;
+    top[e] = on ? a.top[at + 2 * lane + e] : 0.f;
+    in[e] = on ? a.log_i[at + 2 * lane + e] : 0.f;
+  }
   f[1] += f[0];
   double sum = f[1];
 #pragma unroll
@@ -107,8 +113,8 @@ __device__ __forceinline__ void mc_gates(const McArgs& a, const McChunk& m, int 
     A[t] = {0.f, 0.f};
     G[t] = {-INFINITY, 0.f};
     if (t < m.rows) {
-      A[t] = mc_pair(F - (double)a.top[at + t]);
-      G[t] = mc_pair((double)a.log_i[at + t] - F);
+      A[t] = mc_pair(F - (double)top[e]);
+      G[t] = mc_pair((double)in[e] - F);
     }
   }
 }
@@ -174,15 +180,24 @@ __device__ __forceinline__ void mc_store4(__nv_bfloat16* p, __nv_bfloat16 a, __n
   *reinterpret_cast<uint2*>(p) = make_uint2(mc_two(a, b), mc_two(c, d));
 }
 
-// The chunk's rows of one head's `lanes` columns from `col` on as bfloat16, in whole 16s of lanes, zeros behind.
-__device__ __forceinline__ void mc_stage(const McArgs& a, const McChunk& m, int col, int lanes, __nv_bfloat16* to) {
-  const int quads = ((lanes + 15) & ~15) / 4;
-  for (int i = threadIdx.x; i < MC_L * quads; i += blockDim.x) {
-    const int t = i / quads, l = (i - t * quads) * 4;
-    const float4 v = mc_load4(a, (size_t)m.first + t, col, l, lanes, t < m.rows);
-    mc_store4(to + t * MC_PITCH + l, __float2bfloat16_rn(v.x), __float2bfloat16_rn(v.y), __float2bfloat16_rn(v.z),
-              __float2bfloat16_rn(v.w));
+// A block of 256 threads holds a chunk's rows of one head's columns: thread (warp w, lane l) has lanes 4l .. 4l + 3 of the
+// tokens w, w + 8 ...  All of them are asked for before the first is used.
+#define MC_EACH (MC_L / 8)
+__device__ __forceinline__ void mc_fetch(const McArgs& a, const McChunk& m, int col, int lanes, float4 (&v)[MC_EACH]) {
+#pragma unroll
+  for (int j = 0; j < MC_EACH; ++j) {
+    const int t = (threadIdx.x >> 5) + 8 * j;
+    v[j] = mc_load4(a, (size_t)m.first + t, col, (threadIdx.x & 31) * 4, lanes, t < m.rows);
   }
+}
+// As bfloat16 rows in shared memory, in whole 16s of lanes, zeros behind.
+__device__ __forceinline__ void mc_keep(const float4 (&v)[MC_EACH], int lanes, __nv_bfloat16* to) {
+  const int l = (threadIdx.x & 31) * 4;
+  if (l >= ((lanes + 15) & ~15)) return;
+#pragma unroll
+  for (int j = 0; j < MC_EACH; ++j)
+    mc_store4(to + ((threadIdx.x >> 5) + 8 * j) * MC_PITCH + l, __float2bfloat16_rn(v[j].x), __float2bfloat16_rn(v[j].y),
+              __float2bfloat16_rn(v[j].z), __float2bfloat16_rn(v[j].w));
 }
 
 // ---- a chunk's contribution to the state ----
@@ -199,22 +214,27 @@ __global__ void __launch_bounds__(MC_STATE_THREADS) mlstm_chunk_states_kernel(co
   pdl_launch();
   const McChunk m = mc_find(a, blockIdx.x, &found);
   if (m.request < 0) return;
+  float4 v[MC_EACH], keys[MC_EACH];
+  mc_fetch(a, m, a.v_at + head * a.vdim, a.vdim, v);
+  mc_fetch(a, m, a.k_at + head * a.dim, a.dim, keys);
   mc_gates(a, m, head, A, G);
-  mc_stage(a, m, a.v_at + head * a.vdim, a.vdim, v_s);
+  mc_keep(v, a.vdim, v_s);
   __syncthreads();
   const McPair end = A[m.rows - 1];
   const int dk = (a.dim + 15) / 16, dv = (a.vdim + 15) / 16;
-  for (int i = threadIdx.x; i < MC_L * dk * 4; i += MC_STATE_THREADS) {
-    const int t = i / (dk * 4), l = (i - t * dk * 4) * 4;
-    const float4 v = mc_load4(a, (size_t)m.first + t, a.k_at + head * a.dim, l, a.dim, t < m.rows);
-    const float w = mc_exp(end, G[t]);
-    const float x[4] = {v.x, v.y, v.z, v.w};
-    __nv_bfloat16 piece[4][3];
+  if (lane * 4 < dk * 16) {
 #pragma unroll
-    for (int e = 0; e < 4; ++e) mc_split(w * __bfloat162float(__float2bfloat16_rn(x[e])), piece[e]);
+    for (int j = 0; j < MC_EACH; ++j) {
+      const int t = warp + 8 * j;
+      const float w = mc_exp(end, G[t]);
+      const float x[4] = {keys[j].x, keys[j].y, keys[j].z, keys[j].w};
+      __nv_bfloat16 piece[4][3];
 #pragma unroll
-    for (int p = 0; p < 3; ++p)
-      mc_store4(k_s + (p * MC_L + t) * MC_PITCH + l, piece[0][p], piece[1][p], piece[2][p], piece[3][p]);
+      for (int e = 0; e < 4; ++e) mc_split(w * __bfloat162float(__float2bfloat16_rn(x[e])), piece[e]);
+#pragma unroll
+      for (int p = 0; p < 3; ++p)
+        mc_store4(k_s + (p * MC_L + t) * MC_PITCH + lane * 4, piece[0][p], piece[1][p], piece[2][p], piece[3][p]);
+    }
   }
   __syncthreads();
   const size_t cell = (size_t)blockIdx.x * a.heads + head;
@@ -222,7 +242,8 @@ __global__ void __launch_bounds__(MC_STATE_THREADS) mlstm_chunk_states_kernel(co
   if (threadIdx.x == 0) a.decay[cell] = mc_exp(end, {mc_before(a, m, head), 0.f});
   if ((int)threadIdx.x < a.dim) {                       // the normaliser's sum: the weighted keys themselves
     float sum = 0.f;
-    for (int t = 0; t < m.rows; ++t) {
+#pragma unroll 8
+    for (int t = 0; t < MC_L; ++t) {                    // (rows behind the chunk's end are zeros)
       float k = 0.f;
 #pragma unroll
       for (int p = 2; p >= 0; --p) k += __bfloat162float(k_s[(p * MC_L + t) * MC_PITCH + threadIdx.x]);
@@ -281,31 +302,42 @@ __global__ void __launch_bounds__(256) mlstm_chunk_carry_kernel(const McArgs a) 
   const size_t step = (size_t)a.heads * size;
   float* at = a.sums + ((size_t)base * a.heads + head) * size + i;
   const float* decay = a.decay + (size_t)base * a.heads + head;
+  constexpr int DEEP = 8;                                // chunks asked for at once, one batch ahead
+  float sum[2][DEEP][V], d[2][DEEP];
+  auto fetch = [&](int c, int which) {
+#pragma unroll
+    for (int k = 0; k < DEEP; ++k) {
+      if (c + k >= chunks) continue;
+      d[which][k] = decay[(size_t)(c + k) * a.heads];
+      const float* from = at + (c + k) * step;
+      if (V == 2) {
+        const float2 v = *reinterpret_cast<const float2*>(from);
+        sum[which][k][0] = v.x; sum[which][k][1 % V] = v.y;
+      } else {
+        sum[which][k][0] = *from;
+      }
+    }
+  };
+  fetch(0, 0);
   float S[V];
 #pragma unroll
   for (int e = 0; e < V; ++e) S[e] = slot[e];
-  constexpr int DEEP = 8;
-  for (int c = 0; c < chunks; c += DEEP) {
-    float sum[DEEP][V], d[DEEP];
+  auto walk = [&](int c, int which) {
 #pragma unroll
     for (int k = 0; k < DEEP; ++k) {
       if (c + k >= chunks) continue;
-      d[k] = decay[(size_t)(c + k) * a.heads];
-      if (V == 4) {
-        const float4 v = *reinterpret_cast<const float4*>(at + (c + k) * step);
-        sum[k][0] = v.x; sum[k][1 % V] = v.y; sum[k][2 % V] = v.z; sum[k][3 % V] = v.w;
-      } else {
-        sum[k][0] = at[(c + k) * step];
-      }
-    }
+      float* to = at + (c + k) * step;
+      if (V == 2) *reinterpret_cast<float2*>(to) = make_float2(S[0], S[1 % V]);
+      else *to = S[0];
 #pragma unroll
-    for (int k = 0; k < DEEP; ++k) {
-      if (c + k >= chunks) continue;
-      if (V == 4) *reinterpret_cast<float4*>(at + (c + k) * step) = make_float4(S[0], S[1 % V], S[2 % V], S[3 % V]);
-      else at[(c + k) * step] = S[0];
-#pragma unroll
-      for (int e = 0; e < V; ++e) S[e] = fmaf(d[k], S[e], sum[k][e]);
+      for (int e = 0; e < V; ++e) S[e] = fmaf(d[which][k], S[e], sum[which][k][e]);
     }
+  };
+  for (int c = 0; c < chunks; c += 2 * DEEP) {
+    fetch(c + DEEP, 1);
+    walk(c, 0);
+    fetch(c + 2 * DEEP, 0);
+    walk(c + DEEP, 1);
   }
 #pragma unroll
   for (int e = 0; e < V; ++e) slot[e] = S[e];
@@ -334,10 +366,37 @@ __global__ void __launch_bounds__(MC_OUT_THREADS, 2) mlstm_chunk_outputs_kernel(
   const int dk = (a.dim + 15) / 16, dv = (a.vdim + 15) / 16, first_half = (dv + 1) / 2;
   const int my_first = half ? first_half : 0, my_tiles = half ? dv - first_half : first_half;
   const float* S0 = a.sums + ((size_t)blockIdx.x * a.heads + head) * (a.vdim + 1) * a.dim;
-  mc_gates(a, m, head, A, G);
-  mc_stage(a, m, a.q_at + head * a.dim, a.dim, q_s);
-  mc_stage(a, m, a.k_at + head * a.dim, a.dim, k_s);
-  mc_stage(a, m, a.v_at + head * a.vdim, a.vdim, v_s);
+  // a piece of 32 columns of S: thread (warp w, lane l) has lanes 4l .. 4l + 3 of the columns w, w + 8 ..
+  const bool whole4 = (a.dim & 3) == 0;
+  float4 column[4];
+  auto fetch_columns = [&](int j) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int r = warp + 8 * e, l = lane * 4, row = r < 16 ? j * 16 + r : (first_half + j) * 16 + r - 16;
+      column[e] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (row >= a.vdim || l >= a.dim) continue;
+      const float* from = S0 + (size_t)row * a.dim + l;
+      if (whole4) {
+        column[e] = *reinterpret_cast<const float4*>(from);
+      } else {
+        column[e].x = from[0];
+        if (l + 1 < a.dim) column[e].y = from[1];
+        if (l + 2 < a.dim) column[e].z = from[2];
+        if (l + 3 < a.dim) column[e].w = from[3];
+      }
+    }
+  };
+  {
+    float4 rows[MC_EACH];
+    mc_fetch(a, m, a.q_at + head * a.dim, a.dim, rows);
+    fetch_columns(0);
+    mc_gates(a, m, head, A, G);
+    mc_keep(rows, a.dim, q_s);
+    mc_fetch(a, m, a.k_at + head * a.dim, a.dim, rows);
+    mc_keep(rows, a.dim, k_s);
+    mc_fetch(a, m, a.v_at + head * a.vdim, a.vdim, rows);
+    mc_keep(rows, a.vdim, v_s);
+  }
   if (threadIdx.x < 128) norm_s[threadIdx.x] = (int)threadIdx.x < a.dim ? S0[(size_t)a.vdim * a.dim + threadIdx.x] : 0.f;
   const float m0 = mc_before(a, m, head);
   // ---- S_0^T q ----
@@ -346,33 +405,23 @@ __global__ void __launch_bounds__(MC_OUT_THREADS, 2) mlstm_chunk_outputs_kernel(
   for (int j = 0; j < MC_OUT_TILES; ++j)
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[j][0][e] = acc[j][1][e] = 0.f;
-  const bool whole4 = (a.dim & 3) == 0;
 #pragma unroll
   for (int j = 0; j < MC_OUT_TILES; ++j) {
     if (j >= first_half) break;
     if (j) __syncthreads();                             // the pieces before have been read
-    for (int i = threadIdx.x; i < 32 * dk * 4; i += MC_OUT_THREADS) {
-      const int r = i / (dk * 4), l = (i - r * dk * 4) * 4;
-      const int row = (r < 16 ? j * 16 : (first_half + j) * 16 - 16) + r;
-      float x[4] = {0.f, 0.f, 0.f, 0.f};
-      if (row < a.vdim && l < a.dim) {
-        const float* from = S0 + (size_t)row * a.dim + l;
-        if (whole4) {
-          const float4 v = *reinterpret_cast<const float4*>(from);
-          x[0] = v.x; x[1] = v.y; x[2] = v.z; x[3] = v.w;
-        } else {
+    if (lane * 4 < dk * 16) {
 #pragma unroll
-          for (int e = 0; e < 4; ++e)
-            if (l + e < a.dim) x[e] = from[e];
-        }
+      for (int e = 0; e < 4; ++e) {
+        const float x[4] = {column[e].x, column[e].y, column[e].z, column[e].w};
+        __nv_bfloat16 piece[4][3];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) mc_split(x[c], piece[c]);
+#pragma unroll
+        for (int p = 0; p < 3; ++p)
+          mc_store4(S_s + (p * 32 + warp + 8 * e) * MC_PITCH + lane * 4, piece[0][p], piece[1][p], piece[2][p], piece[3][p]);
       }
-      __nv_bfloat16 piece[4][3];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) mc_split(x[e], piece[e]);
-#pragma unroll
-      for (int p = 0; p < 3; ++p)
-        mc_store4(S_s + (p * 32 + r) * MC_PITCH + l, piece[0][p], piece[1][p], piece[2][p], piece[3][p]);
     }
+    if (j + 1 < first_half) fetch_columns(j + 1);
     __syncthreads();
     if (j < my_tiles) {
       for (int k = 0; k < dk; ++k) {
@@ -458,6 +507,22 @@ __global__ void __launch_bounds__(MC_OUT_THREADS, 2) mlstm_chunk_outputs_kernel(
   const float* tops = a.top + (size_t)head * a.gate_ld + m.first;
   const float inv_lo = on_lo ? 1.0f / (fmaxf(fabsf(fmaf(w_lo, den_s[t_lo], own_lo)), expf(-tops[t_lo])) + MC_EPS) : 0.f;
   const float inv_hi = on_hi ? 1.0f / (fmaxf(fabsf(fmaf(w_hi, den_s[t_hi], own_hi)), expf(-tops[t_hi])) + MC_EPS) : 0.f;
+  float2 z[MC_OUT_TILES][2][2];                         // the gate, asked for at once
+  const bool even = ((a.vdim | a.ld | a.g_at) & 1) == 0 && ((uintptr_t)a.proj & 7) == 0;
+#pragma unroll
+  for (int j = 0; j < MC_OUT_TILES; ++j)
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int l = (my_first + j) * 16 + 8 * n + 2 * q;
+        z[j][n][h] = make_float2(0.f, 0.f);
+        if (j < my_tiles && l < a.vdim && (h ? on_hi : on_lo)) {
+          const float* from = a.proj + (size_t)(m.first + (h ? t_hi : t_lo)) * a.ld + a.g_at + head * a.vdim + l;
+          if (even) z[j][n][h] = *reinterpret_cast<const float2*>(from);
+          else z[j][n][h] = make_float2(from[0], l + 1 < a.vdim ? from[1] : 0.f);
+        }
+      }
   float sq_lo = 0.f, sq_hi = 0.f;
 #pragma unroll
   for (int j = 0; j < MC_OUT_TILES; ++j)
@@ -492,15 +557,15 @@ __global__ void __launch_bounds__(MC_OUT_THREADS, 2) mlstm_chunk_outputs_kernel(
       for (int h = 0; h < 2; ++h) {
         const int t = h ? t_hi : t_lo;
         if (!(h ? on_hi : on_lo)) continue;
-        const float* z = a.proj + (size_t)(m.first + t) * a.ld + a.g_at + head * a.vdim + l;
         __nv_bfloat16* o = a.out + ((size_t)(m.first + t) * a.heads + head) * a.vdim + l;
         const float inv = h ? r_hi : r_lo;
-        const float v0 = acc[j][n][2 * h] * inv * g0 / (1.0f + expf(-z[0]));
+        const float v0 = acc[j][n][2 * h] * inv * g0 / (1.0f + expf(-z[j][n][h].x));
+        const float v1 = acc[j][n][2 * h + 1] * inv * g1 / (1.0f + expf(-z[j][n][h].y));
         if (two && (a.vdim & 1) == 0) {
-          *reinterpret_cast<__nv_bfloat162*>(o) = __floats2bfloat162_rn(v0, acc[j][n][2 * h + 1] * inv * g1 / (1.0f + expf(-z[1])));
+          *reinterpret_cast<__nv_bfloat162*>(o) = __floats2bfloat162_rn(v0, v1);
         } else {
           o[0] = __float2bfloat16_rn(v0);
-          if (two) o[1] = __float2bfloat16_rn(acc[j][n][2 * h + 1] * inv * g1 / (1.0f + expf(-z[1])));
+          if (two) o[1] = __float2bfloat16_rn(v1);
         }
       }
     }
@@ -548,8 +613,8 @@ TOKB200_API int tokb200_mlstm_chunks(const float* proj, int ld, int q_at, int k_
   status = launch_dependent(mlstm_chunk_states_kernel, grid, dim3(MC_STATE_THREADS), MC_STATE_SMEM, stream, a);
   if (status != TOKB200_OK) return status;
   const int size = (vdim + 1) * dim;
-  if (dim % 4 == 0 && stride % 4 == 0)
-    status = launch_dependent(mlstm_chunk_carry_kernel<4>, dim3((size / 4 + 255) / 256, heads, n_requests), dim3(256), 0, stream, a);
+  if (size % 2 == 0)
+    status = launch_dependent(mlstm_chunk_carry_kernel<2>, dim3((size / 2 + 255) / 256, heads, n_requests), dim3(256), 0, stream, a);
   else
     status = launch_dependent(mlstm_chunk_carry_kernel<1>, dim3((size + 255) / 256, heads, n_requests), dim3(256), 0, stream, a);
   if (status != TOKB200_OK) return status;

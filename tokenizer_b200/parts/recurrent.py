@@ -415,9 +415,10 @@ class Mamba2:
         return self.out.forward(gated, partials_ok=True)
 
 
-# A step whose longest portion has this many tokens runs the matrix memory in chunks (bfloat16); TOKB200_MEMORY_CHUNKS=0
-# keeps every portion on the scan
-MEMORY_CHUNKS_FROM = 64
+# A step whose longest portion has this many tokens runs the matrix memory in chunks (bfloat16; gates, scan and output
+# norm of a lone request, 16 heads of 128 x 128, us on the scan / in chunks: 64 tokens 23 / 35, 128 43 / 37, 512 72 / 45,
+# 2,048 237 / 95); TOKB200_MEMORY_CHUNKS=0 keeps every portion on the scan
+MEMORY_CHUNKS_FROM = 128
 _MEMORY_CHUNKS = os.environ.get("TOKB200_MEMORY_CHUNKS", "1") != "0"
 
 
