@@ -11,6 +11,7 @@
 #include "common.cuh"
 
 #define ST_MAX 8
+#define ST_PLANES 4
 #define ST_CHUNKS 2            // pieces of a row whose u stays in registers between the sum and the scaling
 
 struct StArgs {
@@ -69,7 +70,9 @@ __device__ __forceinline__ void st_store(__nv_bfloat16* p, const StVec<V>& a) {
   }
 }
 
-template <int STREAMS, int V, typename TO>
+// CUT: y comes as partial sums, of which a few planes are asked for at once (steps of few rows; a whole y keeps the
+// registers that those take for more blocks a multiprocessor).
+template <int STREAMS, int V, bool CUT, typename TO>
 __global__ void __launch_bounds__(512) streams_step_kernel(const StArgs a, TO* __restrict__ out) {
   __shared__ float scratch[33];
   // the weights are written by no kernel of the step: asked for before the wait on the predecessor
@@ -102,10 +105,17 @@ __global__ void __launch_bounds__(512) streams_step_kernel(const StArgs a, TO* _
         y = st_load<V>((const __nv_bfloat16*)a.y + (size_t)t * H + i);
       } else {
         y = st_load<V>((const float*)a.y + (size_t)t * H + i);
-        for (int k = 1; k < a.y_partials; ++k) {
-          const StVec<V> part = st_load<V>((const float*)a.y + (size_t)k * a.y_stride + (size_t)t * H + i);
+        for (int k = 1; CUT && k < a.y_partials; k += ST_PLANES) {      // a few planes asked for at once, added in index order
+          StVec<V> part[ST_PLANES];
 #pragma unroll
-          for (int e = 0; e < V; ++e) y.v[e] += part.v[e];
+          for (int d = 0; d < ST_PLANES; ++d)
+            if (k + d < a.y_partials) part[d] = st_load<V>((const float*)a.y + (size_t)(k + d) * a.y_stride + (size_t)t * H + i);
+#pragma unroll
+          for (int d = 0; d < ST_PLANES; ++d) {
+            if (k + d >= a.y_partials) continue;
+#pragma unroll
+            for (int e = 0; e < V; ++e) y.v[e] += part[d].v[e];
+          }
         }
       }
 #pragma unroll
@@ -190,9 +200,11 @@ static int st_launch(const StArgs& a, void* out, bool quads, cudaStream_t stream
   const int items = quads ? a.hidden / 4 : a.hidden;
   int threads = (items + 31) / 32 * 32;
   threads = threads > 512 ? 512 : threads;
-  if (quads)
-    return launch_dependent(streams_step_kernel<STREAMS, 4, TO>, dim3(a.n_rows), dim3(threads), 0, stream, a, (TO*)out);
-  return launch_dependent(streams_step_kernel<STREAMS, 1, TO>, dim3(a.n_rows), dim3(threads), 0, stream, a, (TO*)out);
+  const dim3 grid(a.n_rows), block(threads);
+  if (quads && a.y && a.y_partials > 1)
+    return launch_dependent(streams_step_kernel<STREAMS, 4, true, TO>, grid, block, 0, stream, a, (TO*)out);
+  if (quads) return launch_dependent(streams_step_kernel<STREAMS, 4, false, TO>, grid, block, 0, stream, a, (TO*)out);
+  return launch_dependent(streams_step_kernel<STREAMS, 1, true, TO>, grid, block, 0, stream, a, (TO*)out);
 }
 
 // x: [T, H] (`equal` not 0: all streams are this one) or [T, streams, H].  y, x_out, read, gain, out and rows may be null
