@@ -1908,7 +1908,7 @@ def run_kerudra(args):
         state, where = torch.zeros(requests, slot, device=dev), f"{T} tokens of {requests} request(s)"
         record(f"mlstm_gates, {where}, {heads} heads",
                kernel_time(lambda: ops.mlstm_gates(proj, at["i"], at["i"] + heads, ib, fb, 15.0, heads, state, m_off, spans, slots, gates)),
-               T * heads * 20, "gdn_prepare")
+               T * heads * 20, None)
         record(f"mlstm_scan, {where}, {heads} heads of {dim} x {vdim}",
                kernel_time(lambda: ops.mlstm_scan(proj, at["q"], at["k"], at["v"], heads, dim, vdim, gates, state, spans, slots, y32, yn)),
                T * heads * (2 * dim + 2 * vdim) * 4, "mamba2_scan", flops=T * heads * dim * (vdim + 1) * 6)

@@ -196,19 +196,21 @@ def linear_bf16_activated(a: torch.Tensor, weight: torch.Tensor, bias: Optional[
     48 / 54, 2,048 rows 76 / 76, 8,192 rows 222 / 199).  TOKB200_GEMM=own keeps every product on the own kernels."""
     M, K = a.shape
     N = weight.shape[0]
-    out = torch.empty((M, N), dtype=torch.bfloat16, device=a.device)
-    if ops._RING and M <= ops.RING_MAX_ROWS and (N * K >= ops.RING_ELEMENTS or M > ops.SMALL_M_ROWS) and \
-            ops.linear_ring_supported(M, N, K, 1):
-        ops.linear_ring(a, weight, bias, out, 1, activation)
-        return out
-    if ops.linear_small_m_supported(M, K) and (M <= ops.SMALL_M_ROWS or N < 4096):
-        ops.linear_small_m(a, weight, bias, out, 1, activation)
-        return out
     choice = os.environ.get("TOKB200_GEMM", "")
-    if ops.gemm_tcgen05_supported(M, N, K) and N % 8 == 0 and choice != "library" and (M >= ACTIVATED_ROWS or choice == "own"):
-        if ops._PAIR and M >= 256:
-            ops.gemm_tcgen05_pair(a, weight, bias, out, ops.PAIR_PLAIN, activation)
-        else:
-            ops.gemm_tcgen05(a, weight, bias, out, activation=activation)
-        return out
-    return ops.activate(linear_bf16(a, weight, bias, torch.bfloat16), activation)
+    ring = ops._RING and M <= ops.RING_MAX_ROWS and (N * K >= ops.RING_ELEMENTS or M > ops.SMALL_M_ROWS) and \
+            ops.linear_ring_supported(M, N, K, 1)
+    few = ops.linear_small_m_supported(M, K) and (M <= ops.SMALL_M_ROWS or N < 4096)
+    tiles = ops.gemm_tcgen05_supported(M, N, K) and N % 8 == 0 and choice != "library" and \
+        (M >= ACTIVATED_ROWS or choice == "own")
+    if not (ring or few or tiles):
+        return ops.activate(linear_bf16(a, weight, bias, torch.bfloat16), activation)
+    out = torch.empty((M, N), dtype=torch.bfloat16, device=a.device)
+    if ring:
+        ops.linear_ring(a, weight, bias, out, 1, activation)
+    elif few:
+        ops.linear_small_m(a, weight, bias, out, 1, activation)
+    elif ops._PAIR and M >= 256:
+        ops.gemm_tcgen05_pair(a, weight, bias, out, ops.PAIR_PLAIN, activation)
+    else:
+        ops.gemm_tcgen05(a, weight, bias, out, activation=activation)
+    return out
