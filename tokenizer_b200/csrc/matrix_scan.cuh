@@ -1,5 +1,5 @@
 // A linear recurrence over a matrix per head, in 32-bit, token by token:
-//     S <- keep S + add b x^T;   y = scale S^T c + skip x
+//     S <- keep S + add b x^T;   y = S^T c + skip x, or scale S^T c
 // with S [N, P] (a request's state, kept as [P, N]), b and c the token's vectors over N (of the head's group of
 // heads), x its vector over P, `keep` and `add` two numbers a token and head.  The mixers that run on it differ in
 // where the two numbers come from and in what their columns are; both are parameters of this kernel.
@@ -37,8 +37,8 @@ struct MatrixScanArgs {
   int P, copied;             // columns, and how many of them x has (P - copied is 0, or 1: the column of ones)
   int N;
   int by16;                  // every row above starts and ends on 16 bytes (set by the launcher)
-  float scale;
-  const float* skip;         // one a head, or null
+  float scale;               // GATES GIVEN: y = scale S^T c
+  const float* skip;         // GATES STEP: y = S^T c + skip x, one a head
   float* state;              // [slots, stride], a slot's matrices [heads, P, N] at its start
   long long stride;
   const int* q_start;
@@ -93,13 +93,15 @@ matrix_scan_kernel(const MatrixScanArgs args) {
   __shared__ __align__(16) float xs[2][RUN][MS_COLS];
   __shared__ float dts[2][RUN];
   __shared__ float decs[2][RUN];
-  const int head = blockIdx.y, r = PASS == 0 ? blockIdx.z : blockIdx.z / segments;
-  const int seg = PASS == 0 ? 0 : blockIdx.z % segments;
+  // neither launch of the two has blocks for a segment that is nothing to it (the last one; the first one): blocks that
+  // end at once would leave the others unevenly spread over the device
+  const int head = blockIdx.y, r = PASS == 0 ? blockIdx.z : blockIdx.z / (segments - 1);
+  const int seg = PASS == 0 ? 0 : blockIdx.z % (segments - 1) + (PASS == 2 ? 1 : 0);
   const int col0 = blockIdx.x * MS_COLS;
   const int part = threadIdx.x % MS_PARTS, mine_x = (threadIdx.x / MS_PARTS) * MS_OWN, col = col0 + mine_x;
   const int group = head / (heads / args.groups);
   const float a = GATES == MS_GATES_STEP ? expf(args.a_log[head]) : 0.f, bias = GATES == MS_GATES_STEP ? args.bias[head] : 0.f;
-  const float d = args.skip ? args.skip[head] : 0.f, scale = args.scale;
+  const float d = GATES == MS_GATES_STEP ? args.skip[head] : 0.f, scale = args.scale;
   // lanes that no copy reaches (rows from N on, columns from P on) stay zero in both halves
   if (N < NPER * MS_PARTS) {
     for (int i = threadIdx.x; i < 2 * RUN * NPAD; i += MS_THREADS) {
@@ -112,7 +114,9 @@ matrix_scan_kernel(const MatrixScanArgs args) {
     for (int i = threadIdx.x; i < 2 * RUN * MS_COLS; i += MS_THREADS)
       (&xs[0][0][0])[i] = (P > copied && i % MS_COLS == copied - col0) ? 1.f : 0.f;
   pdl_wait();
-  pdl_launch();
+  // the second launch of the two starts when the first one's blocks end: blocks that came earlier would take whatever
+  // places the first has left and lie unevenly (8,192 tokens of a lone request: 1.22 against 1.42 ms)
+  if (PASS != 1) pdl_launch();
   int first = args.q_start[r], n = args.q_start[r + 1] - first;
   if (n <= 0) return;
   float* mine = state + (size_t)args.state_slot[r] * stride + ((size_t)head * P + col) * N;
@@ -191,7 +195,6 @@ matrix_scan_kernel(const MatrixScanArgs args) {
         if (blockIdx.x == 0 && threadIdx.x == 0) product = products + (size_t)seg * heads;
       }
     } else {
-      if (seg == 0) return;
       load(ends, S);
       for (int j = 1; j < seg; ++j) {
         float2 local[MS_OWN][NPER / 2];
@@ -209,9 +212,11 @@ matrix_scan_kernel(const MatrixScanArgs args) {
   __syncthreads();                         // the zeros are written before the first copies land
   // 16 bytes a copy where rows, lanes and channels come in whole 4s (a piece of 4 rows lies inside one part)
   const bool by16 = args.by16 != 0;
-  const float* const b_base = args.b + (size_t)group * args.b_group;
-  const float* const c_base = args.c + (size_t)group * args.c_group;
-  const float* const x_base = args.x + (size_t)head * args.x_head + col0;
+  const float* __restrict__ const b_base = args.b + (size_t)group * args.b_group;
+  const float* __restrict__ const c_base = args.c + (size_t)group * args.c_group;
+  const float* __restrict__ const x_base = args.x + (size_t)head * args.x_head + col0;
+  const size_t y_ld = (size_t)heads * copied;
+  float* __restrict__ const y_base = args.y + (size_t)first * y_ld + (size_t)head * copied;
   auto stage = [&](int run, int half) {    // the copies of a run's x, b and c, in flight when it returns
     const int here = n - run < RUN ? n - run : RUN;
     const int cols = copied - col0 < MS_COLS ? copied - col0 : MS_COLS;
@@ -269,9 +274,8 @@ matrix_scan_kernel(const MatrixScanArgs args) {
     }
   };
   auto write = [&](int token, int column, float x, float sum) {
-    const size_t t = (size_t)(first + token);
-    if (column < copied) args.y[(t * heads + head) * copied + column] = fmaf(d, x, scale * sum);
-    else if (column < P) args.y_ones[t * heads + head] = scale * sum;
+    if (column < copied) y_base[token * y_ld + column] = GATES == MS_GATES_STEP ? fmaf(d, x, sum) : scale * sum;
+    else if (GATES == MS_GATES_GIVEN && column < P) args.y_ones[(size_t)(first + token) * heads + head] = scale * sum;
   };
   float decayed = 1.f;                     // the product of the decays of a run from zero
   stage(0, 0);
@@ -395,7 +399,7 @@ static int launch_matrix_scan(MatrixScanArgs a, cudaStream_t stream) {
     return TOKB200_BAD_SIZE;
   a.by16 = ((a.N | a.copied | a.x_ld | a.x_head | a.b_ld | a.b_group | a.c_ld | a.c_group) & 3) == 0 &&
            (((uintptr_t)a.x | (uintptr_t)a.b | (uintptr_t)a.c) & 15) == 0;
-  const dim3 grid((a.P + MS_COLS - 1) / MS_COLS, a.heads, a.n_requests * a.segments);
+  const dim3 grid((a.P + MS_COLS - 1) / MS_COLS, a.heads, a.n_requests * (a.segments > 1 ? a.segments - 1 : 1));
 #define MS_LAUNCH_PASS(NPER, PASS) launch_dependent(matrix_scan_kernel<NPER, TI, GATES, PASS>, grid, dim3(MS_THREADS), 0, stream, a)
 #define MS_LAUNCH(NPER)                                             \
   {                                                                 \
